@@ -7,8 +7,9 @@ from .zurolorn import ZurolornConfig    # registers Zurolorn
 from .ronolorn import RonolornConfig    # registers Ronolorn
 from .gipozen import GipozenConfig      # registers Gipozen
 from .vilodra import VilodraConfig      # registers Vilodra
+from .kezunex import KezunexConfig      # registers Kezunex
 from .presets import preset, preset_dict, preset_names
 
-__all__ = ["CacheUse", "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "LlamaConfig", "ZurolornConfig", "RonolornConfig", "GipozenConfig", "VilodraConfig",
+__all__ = ["CacheUse", "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "LlamaConfig", "ZurolornConfig", "RonolornConfig", "GipozenConfig", "VilodraConfig", "KezunexConfig",
            "ARCHITECTURES", "Architecture", "architecture_for", "register_architecture",
            "preset", "preset_dict", "preset_names"]

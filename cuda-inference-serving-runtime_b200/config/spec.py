@@ -49,11 +49,13 @@ class RunEntry:
     `layer` indexes `ModelSpec.layers`; naming a layer twice runs its weights
     twice.  Each entry owns a cache of its own unless `cache_of` names an earlier
     entry, whose cache it then reads without writing.  `pass_step` t: row t of the model's per-pass vectors
-    (`ModelSpec.pass_steps`) is added to the residual stream right before this entry runs.
+    (`ModelSpec.pass_steps`) is added to the residual stream right before this entry runs.  `add_embedding`: the embedding
+    output (the stream as it was before the first entry) is added there too, first (streams that keep it: "post_norm").
     """
     layer: int
     cache_of: Optional[int] = None
     pass_step: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -107,6 +109,8 @@ class ModelSpec:
                 raise ValueError(f"run entry {i} names layer {entry.layer}, which does not exist")
             if entry.pass_step is not None and self.pass_steps is None:
                 raise ValueError(f"run entry {i} names a per-pass vector, but the model has none")
+            if entry.add_embedding and not self.stream.get("keep_embedding", False):
+                raise ValueError(f"run entry {i} adds the embedding output again, but the residual stream does not keep it")
             if entry.cache_of is not None:
                 if not 0 <= entry.cache_of < i:
                     raise ValueError(f"run entry {i} reads the cache of entry {entry.cache_of}, which must run earlier")

@@ -3,8 +3,10 @@
 // kernels are built for, keys and values written into their cache pages.
 //
 //   row   = proj[t] + bias                                   (bias null: none)
-//   qn    = q_norm ? q / sqrt(mean(q^2) + eps) * q_norm : q  (the mean runs over ALL query heads of the token at once)
+//   qn    = q_norm ? q / sqrt(mean(q^2) + eps) * q_norm : q  (the mean runs over ALL query heads of the token at once, or,
+//           per_head, over each head by itself with one weight of key_dim numbers for all of them)
 //   kn    = k_norm ? k / sqrt(mean(k^2) + eps) * k_norm : k
+//   qn    *= 1 + temp_coef ln(floor((position + 1) / temp_every) + 1)           (temp_coef 0: as it is)
 //   q_out[t][h] = [rotate(qn_h) | 0]                          (key_dim wide, padded with zeros to D)
 //   k_cache[page][g][off] = [rotate(kn_g) | 0]
 //   v_cache[page][g][off] = [v_g | 0]  with v from its own columns, or (v_col < 0) the key as projected: with its bias,
@@ -55,7 +57,7 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
                       QT* __restrict__ q_out, CT* __restrict__ k_cache, CT* __restrict__ v_cache,
                       const int* __restrict__ token_req, const int* __restrict__ positions, const int* __restrict__ req_slot,
                       const int* __restrict__ block_table, int table_width, int page_size, int hq, int hkv, int key_dim,
-                      int value_dim, int D, int n_cols) {
+                      int value_dim, int D, int n_cols, int per_head, float temp_coef, double temp_every) {
     extern __shared__ float row[];            // n_cols floats: the token's projection with its bias
     __shared__ float scratch[32];
     pdl_trigger();
@@ -68,12 +70,12 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
     __syncthreads();
     const int nq = hq * key_dim, nk = hkv * key_dim;
     float inv_q = 1.f, inv_k = 1.f;
-    if (q_norm) {
+    if (q_norm && !per_head) {
         float sq = 0.f;
         for (int i = threadIdx.x; i < nq; i += blockDim.x) sq += row[i] * row[i];
         inv_q = 1.f / sqrtf(block_sum(sq, scratch) / (float)nq + eps);
     }
-    if (k_norm) {
+    if (k_norm && !per_head) {
         float sq = 0.f;
         for (int i = threadIdx.x; i < nk; i += blockDim.x) sq += row[k_col + i] * row[k_col + i];
         inv_k = 1.f / sqrtf(block_sum(sq, scratch) / (float)nk + eps);
@@ -82,22 +84,32 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
     const float* sn = sin_t ? sin_t + (size_t)t * rot_half : nullptr;
     // a warp per head, a lane per pair of neighbouring coordinates (D is even: pairs never straddle heads)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
-    for (int h = warp; h < hq; h += n_warps)
+    const auto head_inv = [&](const float* head) {      // a head's own root mean square (the whole warp takes part)
+        float sq = 0.f;
+        for (int d = lane; d < key_dim; d += 32) sq += head[d] * head[d];
+        return 1.f / sqrtf(warp_sum(sq) / (float)key_dim + eps);
+    };
+    const float temp = temp_coef != 0.f ? 1.f + temp_coef * logf((float)(floor((double)(pos + 1) / temp_every) + 1.0)) : 1.f;
+    for (int h = warp; h < hq; h += n_warps) {
+        const float inv = temp * (q_norm && per_head ? head_inv(row + h * key_dim) : inv_q);
+        const float* w = q_norm ? q_norm + (per_head ? 0 : h * key_dim) : nullptr;
         for (int d = 2 * lane; d < D; d += 64)
-            store_pair(q_out + ((size_t)t * hq + h) * D + d,
-                       turned_pair(row + h * key_dim, q_norm ? q_norm + h * key_dim : nullptr, inv_q, d, key_dim, rot_half, interleaved, cs, sn));
+            store_pair(q_out + ((size_t)t * hq + h) * D + d, turned_pair(row + h * key_dim, w, inv, d, key_dim, rot_half, interleaved, cs, sn));
+    }
     if (!k_cache) return;
     const int page = block_table[(size_t)slot * table_width + pos / page_size];
     if (page < 0) return;                     // the host reserves a page before every write; never follow a missing entry
     const int off = pos % page_size;
-    for (int g = warp; g < hkv; g += n_warps)
+    for (int g = warp; g < hkv; g += n_warps) {
+        const float inv = k_norm && per_head ? head_inv(row + k_col + g * key_dim) : inv_k;
+        const float* w = k_norm ? k_norm + (per_head ? 0 : g * key_dim) : nullptr;
         for (int d = 2 * lane; d < D; d += 64) {
             const float* vs = v_col >= 0 ? row + v_col + g * value_dim : row + k_col + g * key_dim;
             const size_t dst = (((size_t)page * hkv + g) * page_size + off) * D + d;
-            store_pair(k_cache + dst, turned_pair(row + k_col + g * key_dim, k_norm ? k_norm + g * key_dim : nullptr, inv_k, d, key_dim,
-                                                  rot_half, interleaved, cs, sn));
+            store_pair(k_cache + dst, turned_pair(row + k_col + g * key_dim, w, inv, d, key_dim, rot_half, interleaved, cs, sn));
             store_pair(v_cache + dst, make_float2(d < value_dim ? vs[d] : 0.f, d + 1 < value_dim ? vs[d + 1] : 0.f));
         }
+    }
 }
 
 // out[t][c] += bias[c]
@@ -112,11 +124,12 @@ CISR_EXPORT int cisr_attention_rows(const float* proj, int row_stride, int k_col
                                     int interleaved, void* q_out, int q_dtype, void* k_cache, void* v_cache, int cache_dtype,
                                     const int* token_req, const int* positions, const int* req_slot, const int* block_table,
                                     int table_width, int page_size, int hq, int hkv, int key_dim, int value_dim, int D, int tokens,
-                                    void* stream) {
+                                    int per_head, float temp_coef, double temp_every, void* stream) {
     if (tokens <= 0) return 0;
     if (2 * rot_half > key_dim || rot_half < 0 || key_dim > D || value_dim > D || hq <= 0 || hkv <= 0) return -2;
     if (v_col < 0 && value_dim != key_dim) return -2;
     if (rot_half && (!cos_t || !sin_t)) return -2;
+    if (temp_coef != 0.f && !(temp_every > 0.0)) return -2;
     const int n_cols = v_col >= 0 ? v_col + hkv * value_dim : k_col + hkv * key_dim;
     if (n_cols > row_stride) return -2;
     const size_t smem = sizeof(float) * (size_t)n_cols;
@@ -134,7 +147,8 @@ CISR_EXPORT int cisr_attention_rows(const float* proj, int row_stride, int k_col
         const int threads = (tokens <= 64 && n_cols >= 1024) ? 1024 : 256;                                                \
         return launch_kernel(attention_rows_kernel<QT, CT>, dim3(tokens), dim3(threads), smem, s, g_pdl, proj, row_stride, k_col, v_col, bias, \
                              q_norm, k_norm, eps, cos_t, sin_t, rot_half, interleaved, (QT*)q_out, (CT*)k_cache, (CT*)v_cache,   \
-                             token_req, positions, req_slot, block_table, table_width, page_size, hq, hkv, key_dim, value_dim, D, n_cols); \
+                             token_req, positions, req_slot, block_table, table_width, page_size, hq, hkv, key_dim, value_dim, D, n_cols,     \
+                             per_head, temp_coef, temp_every);                                                                                  \
     } while (0)
     if (q_dtype == CISR_BF16 && cache_dtype == CISR_BF16) CISR_ROWS(__nv_bfloat16, __nv_bfloat16);
     if (q_dtype == CISR_F32 && cache_dtype == CISR_F32) CISR_ROWS(float, float);

@@ -55,6 +55,15 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// gelu in its tanh form, 0.5 z (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), written as z / (1 + exp(-2 u)).
+__device__ __forceinline__ float gelu_tanh(float z) {
+    const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return z / (1.f + expf(-2.f * u));
+}
+
+// Activation of the gate in a gated feed-forward: silu (kind 0) or the tanh form of gelu (kind 1).
+__device__ __forceinline__ float gate_activation(float z, int kind) { return kind == 1 ? gelu_tanh(z) : z / (1.f + expf(-z)); }
+
 // Sum over a whole block in a fixed order (warp shuffles, then warp 0 over the
 // per-warp sums), so a row's result does not depend on what else is in the batch.
 __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floats */) {

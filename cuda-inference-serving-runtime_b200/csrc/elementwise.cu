@@ -246,9 +246,9 @@ CISR_EXPORT int cisr_add_rmsnorm(float* x, const float* delta, const void* weigh
 }
 
 // ---------------------------------------------------------------- SwiGLU
-// gate_up [T, 2I] float: gate in columns [0, I), up in [I, 2I).  out = gate/(1+exp(-gate)) * up.
+// gate_up [T, 2I] float: gate in columns [0, I), up in [I, 2I).  out = act(gate) * up, act silu (gate_act 0) or the tanh form of gelu (1).
 template <typename OT>
-__global__ void swiglu_kernel(const float* __restrict__ gate_up, OT* __restrict__ out, int inter, size_t total) {
+__global__ void swiglu_kernel(const float* __restrict__ gate_up, OT* __restrict__ out, int inter, int gate_act, size_t total) {
     CISR_TRACE_SCOPE(TRACE_SWIGLU);
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
@@ -256,16 +256,16 @@ __global__ void swiglu_kernel(const float* __restrict__ gate_up, OT* __restrict_
     const int c = (int)(i - t * inter);
     const float g = gate_up[t * 2 * inter + c];
     const float u = gate_up[t * 2 * inter + inter + c];
-    out[i] = from_float<OT>(g / (1.f + expf(-g)) * u);
+    out[i] = from_float<OT>(gate_activation(g, gate_act) * u);
 }
 
-CISR_EXPORT int cisr_swiglu(const float* gate_up, void* out, int out_dtype, int tokens, int inter, void* stream) {
+CISR_EXPORT int cisr_swiglu(const float* gate_up, void* out, int out_dtype, int tokens, int inter, int gate_act, void* stream) {
     const size_t total = (size_t)tokens * inter;
     if (!total) return 0;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == CISR_BF16) swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (__nv_bfloat16*)out, inter, total);
-    else swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (float*)out, inter, total);
+    if (out_dtype == CISR_BF16) swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (__nv_bfloat16*)out, inter, gate_act, total);
+    else swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (float*)out, inter, gate_act, total);
     return launch_status();
 }
 

@@ -35,7 +35,7 @@ constexpr int BK = 64, UMMA_K = 16;     // BM = 128 (tcgen05.cuh)
 struct Epilogue {                       // what the epilogue variants need beyond the accumulator
     float* out_f32; bf16* out_bf16; int inter;
     float limit, alpha;                 // GATED: g' = min(g, limit), u' = clamp(u, +-limit), g' sigmoid(alpha g') (u' + 1)
-    int act;                            // RELU2's activation: 0 max(z, 0)^2, 1 the exact gelu z Phi(z)
+    int act;                            // RELU2's activation: 0 max(z, 0)^2, 1 the exact gelu z Phi(z); SWIGLU's gate: 0 silu, 1 the tanh form of gelu
     int accumulate;                     // PLAIN: out += product
     float out_mult;                     // PLAIN: the product is multiplied by it first (a constant factor of the residual branch); 0: no factor (the residual stream, in place) instead of out = product
     const float* cos_t; const float* sin_t; bf16* q_out; bf16* k_cache; bf16* v_cache; const int* positions;
@@ -147,6 +147,8 @@ __device__ __forceinline__ void epilogue_tile(const Epilogue& ep, uint32_t lane_
                 store_bf16x32(ep.out_bf16 + (size_t)row * ep.inter + n0 + c, act, ep.inter - (n0 + c));
         }
     } else if (EPI == EPI_SWIGLU) {
+        // silu(z) = z / (1 + exp(-z)) and gelu(z) = z / (1 + exp(-2 sqrt(2 / pi) (z + 0.044715 z^3))) differ in the exponent only
+        const float lin = ep.act == 1 ? 2.f * 0.7978845608028654f : 1.f, cub = ep.act == 1 ? 0.044715f : 0.f;
 #pragma unroll 1
         for (int c = 0; c < BN / 2; c += 32) {
             uint32_t g[32], u[32];
@@ -156,7 +158,7 @@ __device__ __forceinline__ void epilogue_tile(const Epilogue& ep, uint32_t lane_
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
                 const float gv = __uint_as_float(g[j]);
-                act[j] = gv / (1.f + expf(-gv)) * __uint_as_float(u[j]);
+                act[j] = gv / (1.f + expf(-lin * (gv + cub * gv * gv * gv))) * __uint_as_float(u[j]);
             }
             if (row < m && n0 + c < ep.inter)
                 store_bf16x32(ep.out_bf16 + (size_t)row * ep.inter + n0 + c, act, ep.inter - (n0 + c));
@@ -446,13 +448,14 @@ CISR_EXPORT int cisr_gemm_tcgen05(const void* a, const void* w, float* out, int 
     return launch<128, 3, EPI_PLAIN>(a, w, ep, m, n, k, (n + 127) / 128, s);
 }
 
-// w stacks gate rows [0, inter) over up rows [inter, 2 * inter); out (bfloat16 [m, inter]) = silu(a gate^T) * (a up^T).
-CISR_EXPORT int cisr_gemm_tcgen05_swiglu(const void* a, const void* w, void* out, int m, int inter, int k, void* stream) {
+// w stacks gate rows [0, inter) over up rows [inter, 2 * inter); out (bfloat16 [m, inter]) = act(a gate^T) * (a up^T), act silu (gate_act 0)
+// or the tanh form of gelu (1).
+CISR_EXPORT int cisr_gemm_tcgen05_swiglu(const void* a, const void* w, void* out, int m, int inter, int k, int gate_act, void* stream) {
     if (m <= 0 || inter <= 0) return 0;
     if (!g_encode || !g_error) return -13;
     if (!operands_ok(a, w, k)) return -2;
     Epilogue ep = {};
-    ep.out_bf16 = (bf16*)out; ep.inter = inter;
+    ep.out_bf16 = (bf16*)out; ep.inter = inter; ep.act = gate_act;
     if (wide_tiles(m, (inter + 127) / 128)) {
         // 128 x 256 tiles, or 128 x 192 where their last round would be much emptier: 192 tiles of 256 columns on 148 SMs
         // are two rounds for 1.3 rounds of work, 256 tiles of 192 columns are two rounds of three quarters the length

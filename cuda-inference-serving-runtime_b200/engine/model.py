@@ -106,7 +106,7 @@ class Model:
         """The parts whose launch plans travel with every step's metadata, one per plan key."""
         from .batch import unique_planners
 
-        return unique_planners(part for _, part in self._named_parts())
+        return unique_planners(p for _, part in self._named_parts() for p in part.planning_parts())
 
     def compile_kernels(self) -> None:
         """Build, in parallel, exactly the kernel libraries this model launches."""
@@ -160,6 +160,8 @@ class Model:
             part.begin_step(ctx)
         stream = self.stream_class(self.embedding.forward(ctx.token_ids), self.spec.stream)
         for index, entry in enumerate(self.spec.run):
+            if entry.add_embedding:
+                stream.add_embedding()
             if entry.pass_step is not None:
                 self.pass_steps.add_to(stream, entry.pass_step)
             self.layers[entry.layer].forward(stream, ctx, cache.binding(index, reads_from=entry.cache_of))

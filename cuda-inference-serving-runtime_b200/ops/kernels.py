@@ -155,13 +155,16 @@ def scale_(x: torch.Tensor, scale: float) -> torch.Tensor:
     return x
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out = silu(gate_up[:, :I]) * gate_up[:, I:]."""
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}       # of the gate in a gated feed-forward
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, gate: str = "silu") -> torch.Tensor:
+    """out = act(gate_up[:, :I]) * gate_up[:, I:], act silu or the tanh form of gelu."""
     _need(gate_up, torch.float32, "gate_up", 2); _need(out, None, "out", 2)
     tokens, inter = out.shape
     if gate_up.shape != (tokens, 2 * inter):
         raise KernelError("swiglu: gate_up must be [tokens, 2 * intermediate]")
-    _check(_elementwise().cisr_swiglu(_p(gate_up), _p(out), dtype_code(out.dtype), tokens, inter, _stream()), "swiglu")
+    _check(_elementwise().cisr_swiglu(_p(gate_up), _p(out), dtype_code(out.dtype), tokens, inter, GATE_ACTIVATIONS[gate], _stream()), "swiglu")
     return out
 
 
@@ -782,10 +785,12 @@ def attention_rows(proj: torch.Tensor, k_col: int, v_col: int, *, bias: Optional
                    k_norm: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot_half: int,
                    interleaved: bool, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, token_req: torch.Tensor,
                    positions: torch.Tensor, req_slot: torch.Tensor, block_table: torch.Tensor, page_size: int, hq: int, hkv: int,
-                   key_dim: int, value_dim: int) -> None:
+                   key_dim: int, value_dim: int, norm_per_head: bool = False, q_temp=None) -> None:
     """proj float [tokens, cols] holds q at column 0, k at `k_col`, v at `v_col` (`v_col` < 0: the values are the keys as
-    projected).  Adds `bias` (float [cols]), norms q and k over their whole projection (`q_norm`, `k_norm`: float weights of
-    that size, or None), rotates, pads the heads to the cache's width D, writes q_out [tokens, hq, D] and the key and value
+    projected; columns behind those are another reader's).  Adds `bias` (float [cols]), norms q and k over their whole
+    projection (`q_norm`, `k_norm`: float weights of that size, or None) or, with `norm_per_head`, each head by itself (weights
+    of one head's size, shared by all), multiplies q by 1 + coef * ln(floor((position + 1) / every) + 1) where `q_temp` =
+    (coef, every) is given, rotates, pads the heads to the cache's width D, writes q_out [tokens, hq, D] and the key and value
     rows into their pages ([pages, hkv, page_size, D]).  See csrc/attention_rows.cu."""
     _need(proj, torch.float32, "proj", 2); _need(q_out, None, "q_out", 3); _need(k_cache, q_out.dtype, "k_cache", 4)
     _need(v_cache, q_out.dtype, "v_cache", 4)
@@ -793,7 +798,8 @@ def attention_rows(proj: torch.Tensor, k_col: int, v_col: int, *, bias: Optional
     width = k_cache.shape[-1]
     if tuple(q_out.shape) != (tokens, hq, width) or tuple(k_cache.shape[1:]) != (hkv, page_size, width) or v_cache.shape != k_cache.shape:
         raise KernelError("attention_rows: q_out must be [tokens, hq, D] and the caches [pages, hkv, page_size, D]")
-    for name, t, n in (("bias", bias, cols), ("q_norm", q_norm, hq * key_dim), ("k_norm", k_norm, hkv * key_dim)):
+    for name, t, n in (("bias", bias, cols), ("q_norm", q_norm, key_dim if norm_per_head else hq * key_dim),
+                       ("k_norm", k_norm, key_dim if norm_per_head else hkv * key_dim)):
         if t is not None:
             _need(t, torch.float32, name, 1)
             if t.numel() != n:
@@ -808,7 +814,8 @@ def attention_rows(proj: torch.Tensor, k_col: int, v_col: int, *, bias: Optional
         _p(proj), cols, k_col, v_col, _p(bias), _p(q_norm), _p(k_norm), ctypes.c_float(eps), _p(cos if rot_half else None),
         _p(sin if rot_half else None), rot_half, int(interleaved), _p(q_out), dtype_code(q_out.dtype), _p(k_cache), _p(v_cache),
         dtype_code(k_cache.dtype), _p(token_req), _p(positions), _p(req_slot), _p(block_table), block_table.shape[1], page_size,
-        hq, hkv, key_dim, value_dim, width, tokens, _stream()), "attention_rows")
+        hq, hkv, key_dim, value_dim, width, tokens, int(norm_per_head), ctypes.c_float(q_temp[0] if q_temp else 0.0),
+        ctypes.c_double(q_temp[1] if q_temp else 1.0), _stream()), "attention_rows")
 
 
 def bias_add(out: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
@@ -1003,6 +1010,316 @@ def lightning_output(o: torch.Tensor, gate: torch.Tensor, gate_col: int, norm_w:
         raise KernelError("lightning_output: shapes disagree")
     _check(_lightning().cisr_lightning_output(_p(o), _p(gate), gate.shape[1], gate_col, _p(norm_w), ctypes.c_float(eps), _p(out),
                                               dtype_code(out.dtype), out.shape[1], width, tokens, _stream()), "lightning_output")
+    return out
+
+
+# ------------------------------------------------------------------ norms before and after a sub-block
+_post_norm_state = {}
+
+
+def _loaded(state: dict, source: str, prefix: str, names) -> ctypes.CDLL:
+    """The library `source`, its entry points returning int, told whether launches start early."""
+    lib = state.get("lib")
+    if lib is None:
+        lib = load_library(source)
+        for name in names:
+            getattr(lib, name).restype = ctypes.c_int
+        getattr(lib, f"cisr_{prefix}_set_pdl")(int(_pdl_state["on"]))
+        state["lib"] = lib
+    return lib
+
+
+def post_norm_jobs():
+    return [("post_norm.cu", {}, ())]
+
+
+def post_norm(x: torch.Tensor, *, y: Optional[torch.Tensor] = None, post_w: Optional[torch.Tensor] = None, post_eps: float = 0.0,
+              post_kind: str = "layer", extra: Optional[torch.Tensor] = None, vector: Optional[torch.Tensor] = None,
+              x_out: Optional[torch.Tensor] = None, pre_w: Optional[torch.Tensor] = None, pre_eps: float = 0.0, pre_kind: str = "layer",
+              h: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """v = x + norm(y) * post_w + extra + vector (y, extra, vector: each may be absent); x_out (may be x; None: not
+    stored) receives v, h = norm(v) * pre_w (None: not formed).  Norm kinds: "layer" (mean taken off) or "rms".  `rows` picks
+    rows of x, y and extra that become rows of h (nothing is stored then).  See csrc/post_norm.cu."""
+    _need(x, torch.float32, "x", 2)
+    tokens, hidden = x.shape
+    for name, t, n in (("y", y, 2), ("extra", extra, 2), ("x_out", x_out, 2)):
+        if t is not None:
+            _need(t, torch.float32, name, n)
+            if t.shape != x.shape:
+                raise KernelError(f"post_norm: {name} and x differ in shape")
+    for name, t in (("post_w", post_w if y is not None else None), ("vector", vector), ("pre_w", pre_w if h is not None else None)):
+        if t is not None:
+            _need(t, torch.float32, name, 1)
+            if t.numel() != hidden:
+                raise KernelError(f"post_norm: {name} must have one value per channel")
+    n_rows = tokens
+    if rows is not None:
+        _need(rows, torch.int32, "rows", 1)
+        n_rows = rows.numel()
+        if x_out is not None:
+            raise KernelError("post_norm: rows are picked for reading only")
+    if h is not None:
+        _need(h, None, "h", 2)
+        if h.shape != (n_rows, hidden) or pre_w is None:
+            raise KernelError("post_norm: h must have a row per row read, and needs pre_w")
+    if y is not None and post_w is None:
+        raise KernelError("post_norm: y needs post_w")
+    lib = _loaded(_post_norm_state, "post_norm.cu", "post_norm", ("cisr_post_norm",))
+    _check(lib.cisr_post_norm(_p(x), _p(x_out), _p(y), _p(post_w), ctypes.c_float(post_eps), NORM_KINDS[post_kind], _p(extra), _p(vector),
+                              _p(pre_w), ctypes.c_float(pre_eps), NORM_KINDS[pre_kind], _p(h), dtype_code(h.dtype) if h is not None else 0,
+                              _p(rows), n_rows, hidden, int(x_out is not None), _stream()), "post_norm")
+    return h
+
+
+# ------------------------------------------------------------------ linear recurrence with a matrix state, decays and gains per token
+_gated_state = {}
+GATED_MAX_KEY_DIM = 512
+GATED_CHUNK = 64                 # tokens per chunk of the chunked form; portions of at least this many tokens run chunk by chunk
+
+
+def _gated():
+    fresh = "lib" not in _gated_state
+    lib = _loaded(_gated_state, "gated_linear.cu", "gated", ("cisr_gated_recurrence", "cisr_gated_chunk_tokens", "cisr_gated_max_key_dim"))
+    if fresh:
+        assert lib.cisr_gated_chunk_tokens() == GATED_CHUNK and lib.cisr_gated_max_key_dim() == GATED_MAX_KEY_DIM
+    return lib
+
+
+def gated_jobs():
+    return [("gated_linear.cu", {}, ())]
+
+
+def gated_recurrence(q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: int, v: torch.Tensor, v_col: int, la: torch.Tensor, g: torch.Tensor,
+                     state: torch.Tensor, req_slot: torch.Tensor, q_start: torch.Tensor, q_len: torch.Tensor, n_req: int, y: torch.Tensor,
+                     groups: int, key_dim: int, *, q_scale: float = 1.0, yn: Optional[torch.Tensor] = None, least: int = 0, n_short: int = 0,
+                     chunks=None) -> torch.Tensor:
+    """Per head S <- exp(la) S + g k v^T, y = q_scale * S^T q over each request's tokens in order; with `yn` also n <- exp(la) n +
+    g k, yn = q_scale * n . q.  q, k: float [tokens, columns], `groups` heads of `key_dim` from q_col / k_col (consecutive heads
+    share one); v: heads x dv from v_col; la, g float [tokens, heads]; y float [tokens, heads, dv], yn [tokens, heads].  state
+    float [slots, >= heads * key_dim * (dv, + 1 with yn)] is read and advanced.  `least` > 0 with `chunks` = (chunk_req,
+    chunk_t0, req_chunk0, n_chunks): the requests that bring at least that many tokens run chunk by chunk, the `n_short`
+    others token by token; 0: all token by token.  See csrc/gated_linear.cu."""
+    for name, t, dims in (("q", q, 2), ("k", k, 2), ("v", v, 2), ("la", la, 2), ("g", g, 2), ("state", state, 2), ("y", y, 3)):
+        _need(t, torch.float32, name, dims)
+    for name, t in (("req_slot", req_slot), ("q_start", q_start), ("q_len", q_len)):
+        _need(t, torch.int32, name, 1)
+    tokens, heads, dv = y.shape
+    norm = yn is not None
+    if (la.shape != (tokens, heads) or g.shape != la.shape or heads % groups or key_dim > GATED_MAX_KEY_DIM
+            or q_col + groups * key_dim > q.shape[1] or k_col + groups * key_dim > k.shape[1] or v_col + heads * dv > v.shape[1]
+            or min(q.shape[0], k.shape[0], v.shape[0]) < tokens or state.shape[1] < heads * key_dim * (dv + int(norm))
+            or min(req_slot.numel(), q_start.numel(), q_len.numel()) < n_req):
+        raise KernelError("gated_recurrence: shapes disagree")
+    if norm:
+        _need(yn, torch.float32, "yn", 2)
+        if yn.shape != la.shape:
+            raise KernelError("gated_recurrence: yn must be [tokens, heads]")
+    chunk_req = chunk_t0 = req_chunk0 = scores = blocks = decays = None
+    n_chunks = 0
+    if least > 0 and chunks is not None and chunks[3] > 0:
+        chunk_req, chunk_t0, req_chunk0, n_chunks = chunks
+        for name, t in (("chunk_req", chunk_req), ("chunk_t0", chunk_t0), ("req_chunk0", req_chunk0)):
+            _need(t, torch.int32, name, 1)
+        if chunk_req.numel() < n_chunks or chunk_t0.numel() < n_chunks or req_chunk0.numel() < n_req:
+            raise KernelError("gated_recurrence: the chunk lists are too short")
+        scores = torch.empty((n_chunks, groups, GATED_CHUNK, GATED_CHUNK), dtype=torch.float32, device=y.device)
+        blocks = torch.empty((n_chunks, heads, key_dim * (dv + int(norm))), dtype=torch.float32, device=y.device)
+        decays = torch.empty((n_chunks, heads), dtype=torch.float32, device=y.device)
+    at = lambda t, col: ctypes.c_void_p(t.data_ptr() + 4 * col)
+    _check(_gated().cisr_gated_recurrence(
+        at(q, q_col), q.shape[1], at(k, k_col), k.shape[1], at(v, v_col), v.shape[1], _p(la), _p(g), _p(state), ctypes.c_longlong(state.shape[1]),
+        _p(req_slot), _p(q_start), _p(q_len), _p(y), _p(yn), ctypes.c_float(q_scale), heads, groups, key_dim, dv, n_req,
+        int(least if n_chunks else 0), int(n_chunks), int(n_short), _p(chunk_req), _p(chunk_t0), _p(req_chunk0), _p(scores), _p(blocks),
+        _p(decays), _stream()), "gated_recurrence", own=(4 if n_chunks else 0) + (1 if not n_chunks or n_short else 0))
+    return y
+
+
+# ------------------------------------------------------------------ row kernels around the recurrences
+_recurrent_rows_state = {}
+
+
+def _recurrent_rows():
+    return _loaded(_recurrent_rows_state, "recurrent_rows.cu", "recurrent_rows",
+                   ("cisr_short_conv", "cisr_exp_gates", "cisr_exp_output", "cisr_ssd_output"))
+
+
+def recurrent_rows_jobs():
+    return [("recurrent_rows.cu", {}, ())]
+
+
+def short_conv(proj: torch.Tensor, col: int, taps_w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, keep_offset: int, *,
+               req_slot, q_start, q_len, tile_req, tile_t0, n_tiles: int, tile: int, out: torch.Tensor, silu: bool,
+               in_bias: Optional[torch.Tensor] = None, steps=None, split: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out[t] = act(bias + sum_j taps_w[n - 1 - j] * input(t - j)) per channel, input(t) = proj[t, col:] + in_bias inside the
+    portion and the request's kept inputs before it; then the last taps - 1 inputs become the kept ones (in `state`, float
+    [slots, ...], from `keep_offset`: [taps - 1, channels]).  taps_w float [taps, channels], the last row the current
+    token's; out float [tokens, channels]; tile_req / tile_t0: the step's tokens in tiles of at most `tile` per request.
+    `steps` = (dt_col, dt_bias, a_log, la, g): also dt = softplus(proj[:, dt_col:] + dt_bias), la = -exp(a_log) dt, g = dt, both
+    float [tokens, heads].  `split` bfloat16 [blocks, rows, 3, channels / blocks]: out also as three summands."""
+    _need(proj, torch.float32, "proj", 2); _need(taps_w, torch.float32, "taps_w", 2); _need(state, torch.float32, "state", 2)
+    _need(out, torch.float32, "out", 2)
+    taps, channels = taps_w.shape
+    for name, t in (("bias", bias), ("in_bias", in_bias)):
+        if t is not None:
+            _need(t, torch.float32, name, 1)
+            if t.numel() != channels:
+                raise KernelError(f"short_conv: {name} must have one value per channel")
+    for name, t in (("req_slot", req_slot), ("q_start", q_start), ("q_len", q_len), ("tile_req", tile_req), ("tile_t0", tile_t0)):
+        _need(t, torch.int32, name, 1)
+    if (col + channels > proj.shape[1] or out.shape != (proj.shape[0], channels) or keep_offset + (taps - 1) * channels > state.shape[1]
+            or tile < max(taps - 1, 1) or min(tile_req.numel(), tile_t0.numel()) < n_tiles):
+        raise KernelError("short_conv: shapes disagree")
+    dt_col, dt_bias, a_log, la, g = steps if steps is not None else (0, None, None, None, None)
+    heads = 0
+    if steps is not None:
+        heads = dt_bias.numel()
+        for name, t, dims in (("dt_bias", dt_bias, 1), ("a_log", a_log, 1), ("la", la, 2), ("g", g, 2)):
+            _need(t, torch.float32, name, dims)
+        if dt_col + heads > proj.shape[1] or a_log.numel() != heads or la.shape != (proj.shape[0], heads) or g.shape != la.shape:
+            raise KernelError("short_conv: the step sizes' shapes disagree")
+    if split is not None:
+        _need(split, torch.bfloat16, "split", 4)
+        if split.shape[0] * split.shape[3] != channels or split.shape[2] != 3 or split.shape[1] < proj.shape[0]:
+            raise KernelError("short_conv: split must be [blocks, rows, 3, channels / blocks]")
+    _check(_recurrent_rows().cisr_short_conv(
+        _p(proj), proj.shape[1], col, _p(in_bias), _p(taps_w), _p(bias), taps, channels, int(silu), _p(state), ctypes.c_longlong(state.shape[1]),
+        ctypes.c_longlong(keep_offset), _p(req_slot), _p(q_start), _p(q_len), _p(tile_req), _p(tile_t0), n_tiles, tile, _p(out), dt_col, heads,
+        _p(dt_bias), _p(a_log), _p(la), _p(g), _p(split), split.shape[3] if split is not None else 0,
+        ctypes.c_longlong(split.shape[1] if split is not None else 0), _stream()), "short_conv")
+    return out
+
+
+def exp_gates(proj: torch.Tensor, i_col: int, f_col: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, state: torch.Tensor,
+              m_offset: int, req_slot, q_start, q_len, n_req: int, la: torch.Tensor, g: torch.Tensor, m: torch.Tensor, longest: int = 1 << 30) -> None:
+    """Per token and head, i = cap tanh((proj[:, i_col:] + i_bias) / cap), f = logsigmoid of the like, and with the request's
+    running maximum (state [slots, ...], one float per head from `m_offset`): m = max(f + m_before, i), la = f + m_before - m,
+    g = exp(i - m), all float [tokens, heads].  `longest`: a bound on the portions, for the launch shape only."""
+    for name, t, dims in (("proj", proj, 2), ("i_bias", i_bias, 1), ("f_bias", f_bias, 1), ("state", state, 2), ("la", la, 2), ("g", g, 2), ("m", m, 2)):
+        _need(t, torch.float32, name, dims)
+    heads = i_bias.numel()
+    if (f_bias.numel() != heads or max(i_col, f_col) + heads > proj.shape[1] or la.shape != (proj.shape[0], heads) or g.shape != la.shape
+            or m.shape != la.shape or m_offset + heads > state.shape[1]):
+        raise KernelError("exp_gates: shapes disagree")
+    _check(_recurrent_rows().cisr_exp_gates(_p(proj), proj.shape[1], i_col, f_col, _p(i_bias), _p(f_bias), ctypes.c_float(cap), _p(state),
+                                            ctypes.c_longlong(state.shape[1]), ctypes.c_longlong(m_offset), _p(req_slot), _p(q_start),
+                                            _p(q_len), _p(la), _p(g), _p(m), heads, n_req, int(min(longest, 1 << 30)), _stream()), "exp_gates")
+
+
+def exp_output(y: torch.Tensor, yn: torch.Tensor, m: torch.Tensor, gate: torch.Tensor, gate_col: int, norm_w: torch.Tensor, eps: float,
+               out: torch.Tensor) -> torch.Tensor:
+    """Per head o = y / (max(|yn|, exp(-m)) + 1e-6), o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(gate[:, gate_col:]), rounded to
+    out's type; out may be wider than heads * dv (padding columns are left as they are)."""
+    for name, t, dims in (("y", y, 3), ("yn", yn, 2), ("m", m, 2), ("gate", gate, 2), ("norm_w", norm_w, 1)):
+        _need(t, torch.float32, name, dims)
+    _need(out, None, "out", 2)
+    tokens, heads, dv = y.shape
+    if (yn.shape != (tokens, heads) or m.shape != yn.shape or gate.shape[0] != tokens or gate_col + heads * dv > gate.shape[1]
+            or norm_w.numel() != heads * dv or out.shape[0] != tokens or out.shape[1] < heads * dv):
+        raise KernelError("exp_output: shapes disagree")
+    _check(_recurrent_rows().cisr_exp_output(_p(y), _p(yn), _p(m), _p(gate), gate.shape[1], gate_col, _p(norm_w), ctypes.c_float(eps), _p(out),
+                                             dtype_code(out.dtype), out.shape[1], heads, dv, tokens, _stream()), "exp_output")
+    return out
+
+
+def ssd_output(y: torch.Tensor, x: torch.Tensor, D: torch.Tensor, z: torch.Tensor, z_col: int, norm_w: torch.Tensor, eps: float, out: torch.Tensor,
+               *, parts: int = 1, scale: float = 1.0, lead: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """v = (y + D_h x) silu(z) over a token's row (x: the first heads * dv columns of its tensor, z from z_col), each of `parts`
+    equal parts divided by its root mean square (eps inside), times norm_w and scale, rounded to out's type.  out [tokens, columns]: `lead`
+    (out's type, copied) | v | zeros."""
+    for name, t, dims in (("y", y, 3), ("x", x, 2), ("D", D, 1), ("z", z, 2), ("norm_w", norm_w, 1)):
+        _need(t, torch.float32, name, dims)
+    _need(out, None, "out", 2)
+    tokens, heads, dv = y.shape
+    lead_width = 0
+    if lead is not None:
+        _need(lead, out.dtype, "lead", 2)
+        lead_width = lead.shape[1]
+    if (x.shape[0] != tokens or x.shape[1] < heads * dv or D.numel() != heads or z.shape[0] != tokens or z_col + heads * dv > z.shape[1]
+            or norm_w.numel() != heads * dv or (heads * dv) % parts or out.shape[0] != tokens or out.shape[1] < lead_width + heads * dv
+            or (lead is not None and lead.shape[0] != tokens)):
+        raise KernelError("ssd_output: shapes disagree")
+    _check(_recurrent_rows().cisr_ssd_output(_p(y), _p(x), x.shape[1], _p(D), _p(z), z.shape[1], z_col, _p(norm_w), ctypes.c_float(eps),
+                                             ctypes.c_float(scale), parts, _p(lead), lead_width, _p(out), dtype_code(out.dtype), out.shape[1],
+                                             heads, dv, tokens, _stream()), "ssd_output")
+    return out
+
+
+# ------------------------------------------------------------------ real-gated linear recurrence
+_rglru_state = {}
+RGLRU_FUSED_TOKENS = 16          # steps of at most this many tokens run gates, recurrence and output as one kernel
+
+
+def _rglru():
+    fresh = "lib" not in _rglru_state
+    lib = _loaded(_rglru_state, "rglru.cu", "rglru", ("cisr_rglru_gates", "cisr_rglru_scan", "cisr_rglru_fused_tokens"))
+    if fresh:
+        assert lib.cisr_rglru_fused_tokens() == RGLRU_FUSED_TOKENS
+    return lib
+
+
+def rglru_jobs():
+    return [("rglru.cu", {}, ())]
+
+
+def _rglru_shapes(u, bias, rate, state, s_offset, gate, gate_col, gate_bias, out, blocks: int, what: str) -> tuple:
+    for name, t, dims in (("u", u, 2), ("bias", bias, 2), ("rate", rate, 1), ("state", state, 2), ("gate", gate, 2), ("gate_bias", gate_bias, 1)):
+        if t is not None:
+            _need(t, torch.float32, name, dims)
+    _need(out, None, "out", 2)
+    tokens, width = u.shape
+    block = width // blocks
+    if (width % blocks or (bias is not None and bias.shape != (blocks, 2 * block)) or rate.numel() != width or s_offset + width > state.shape[1]
+            or gate.shape[0] != tokens or gate_col + width > gate.shape[1] or gate_bias.numel() != width or out.shape[0] != tokens
+            or out.shape[1] < width):
+        raise KernelError(f"{what}: shapes disagree")
+    return tokens, width, block
+
+
+def rglru_gates(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, pre: torch.Tensor) -> torch.Tensor:
+    """pre[b, t] = w[b] u_b[t] + bias[b] for the parts of u (float [tokens, width]): w [blocks, 2 block, block] (a part's r rows,
+    then its i rows; any storage type), bias float [blocks, 2 block], pre float [blocks, rows >= tokens, 2 block]."""
+    _need(u, torch.float32, "u", 2); _need(w, None, "w", 3); _need(bias, torch.float32, "bias", 2); _need(pre, torch.float32, "pre", 3)
+    tokens, width = u.shape
+    blocks, two, block = w.shape
+    if blocks * block != width or two != 2 * block or bias.shape != (blocks, two) or pre.shape[0] != blocks or pre.shape[1] < tokens or pre.shape[2] != two:
+        raise KernelError("rglru_gates: shapes disagree")
+    none = ctypes.c_void_p(0)
+    _check(_rglru().cisr_rglru_gates(_p(u), _p(w), dtype_code(w.dtype), _p(bias), _p(pre), ctypes.c_longlong(pre.shape[1]), tokens, width, block, none,
+                                     none, ctypes.c_longlong(0), ctypes.c_longlong(0), none, none, none, none, none, 0, 0, none, none, 0, 0,
+                                     _stream()), "rglru_gates")
+    return pre
+
+
+def rglru_step(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, rate: torch.Tensor, state: torch.Tensor, s_offset: int, token_req, req_slot,
+               q_start, q_len, gate: torch.Tensor, gate_col: int, gate_bias: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """A step of at most RGLRU_FUSED_TOKENS tokens as one kernel: the gates' products, the recurrence over each request's
+    tokens in order (state read and advanced), the output S * gelu(gate + gate_bias) in out's type (the type of w)."""
+    tokens, width, block = _rglru_shapes(u, bias, rate, state, s_offset, gate, gate_col, gate_bias, out, w.shape[0], "rglru_step")
+    _need(w, out.dtype, "w", 3)
+    if tokens > RGLRU_FUSED_TOKENS or w.shape[1:] != (2 * block, block):
+        raise KernelError("rglru_step: too many tokens, or w has the wrong shape")
+    for name, t in (("token_req", token_req), ("req_slot", req_slot), ("q_start", q_start), ("q_len", q_len)):
+        _need(t, torch.int32, name, 1)
+    _check(_rglru().cisr_rglru_gates(_p(u), _p(w), dtype_code(w.dtype), _p(bias), ctypes.c_void_p(0), ctypes.c_longlong(0), tokens, width, block,
+                                     _p(rate), _p(state), ctypes.c_longlong(state.shape[1]), ctypes.c_longlong(s_offset), _p(token_req),
+                                     _p(req_slot), _p(q_start), _p(q_len), _p(gate), gate.shape[1], gate_col, _p(gate_bias), _p(out),
+                                     dtype_code(out.dtype), out.shape[1], _stream()), "rglru_step")
+    return out
+
+
+def rglru_scan(pre: torch.Tensor, bias: Optional[torch.Tensor], u: torch.Tensor, rate: torch.Tensor, state: torch.Tensor, s_offset: int, req_slot,
+               q_start, q_len, n_req: int, gate: torch.Tensor, gate_col: int, gate_bias: torch.Tensor, out: torch.Tensor,
+               longest: int = 1 << 30) -> torch.Tensor:
+    """The recurrence and its output from the gates' sums (pre [blocks, rows, 2 block]; `bias` is added to them, None: they
+    hold it), for portions of any length.  `longest`: a bound on the portions, for the launch shape only."""
+    _need(pre, torch.float32, "pre", 3)
+    tokens, width, block = _rglru_shapes(u, bias, rate, state, s_offset, gate, gate_col, gate_bias, out, pre.shape[0], "rglru_scan")
+    if pre.shape[1] < tokens or pre.shape[2] != 2 * block:
+        raise KernelError("rglru_scan: pre must be [blocks, rows, 2 block]")
+    _check(_rglru().cisr_rglru_scan(_p(pre), ctypes.c_longlong(pre.shape[1]), _p(bias), _p(u), width, block, _p(rate), _p(state),
+                                    ctypes.c_longlong(state.shape[1]), ctypes.c_longlong(s_offset), _p(req_slot), _p(q_start), _p(q_len), _p(gate),
+                                    gate.shape[1], gate_col, _p(gate_bias), _p(out), dtype_code(out.dtype), out.shape[1], n_req,
+                                    int(min(longest, 1 << 30)), _stream()), "rglru_scan")
     return out
 
 
@@ -1455,6 +1772,9 @@ def set_pdl(on: bool) -> None:
         _lightning_state["lib"].cisr_lightning_set_pdl(int(on))
     if "lib" in _diff_state:
         _diff_state["lib"].cisr_diff_set_pdl(int(on))
+    for state, name in ((_post_norm_state, "post_norm"), (_gated_state, "gated"), (_recurrent_rows_state, "recurrent_rows"), (_rglru_state, "rglru")):
+        if "lib" in state:
+            getattr(state["lib"], f"cisr_{name}_set_pdl")(int(on))
     if "lib" in _depth_state:
         _depth_state["lib"].cisr_depth_set_pdl(int(on))
     if "lib" in _ffn_rows_state:
@@ -1496,7 +1816,7 @@ def skinny_gemm(w: torch.Tensor, tokens: int, *, act: Optional[torch.Tensor] = N
                 delta: Optional[torch.Tensor] = None, norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
                 x_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, epilogue: int = EPI_PLAIN,
                 out: Optional[torch.Tensor] = None, rope: Optional[dict] = None, kind: str = "auto",
-                accumulate: bool = False, out_mult: float = 1.0) -> None:
+                accumulate: bool = False, out_mult: float = 1.0, gate: str = "silu") -> None:
     """out = prologue(input) @ w^T with a fused epilogue; see csrc/skinny_gemm.cu and csrc/stream_gemm.cu.
 
     `kind`: "latency" (skinny_gemm.cu: a CTA per 16 output rows, weights straight to registers), "stream"
@@ -1506,7 +1826,8 @@ def skinny_gemm(w: torch.Tensor, tokens: int, *, act: Optional[torch.Tensor] = N
     Input is either `act` (bfloat16 [tokens, K]) or the norm prologue (`x`, optional `delta`, `norm_w`, `eps`,
     optional `x_out` receiving x + delta, optional `rows` picking rows of x).  PLAIN writes float `out`
     [tokens, N], or with `accumulate` adds the product to what `out` holds (the residual stream), in both cases times
-    `out_mult` (a constant factor of the residual branch); SWIGLU writes bfloat16 `out` [tokens, N / 2]; ROPE takes the `rope` dict (cos, sin, rot_half,
+    `out_mult` (a constant factor of the residual branch); SWIGLU writes bfloat16 `out` [tokens, N / 2] with the activation
+    `gate` ("silu" or "gelu_tanh") on the gate; ROPE takes the `rope` dict (cos, sin, rot_half,
     interleaved, q_out, k_cache, v_cache, positions, token_req, req_slot, block_table, page_size, hq, hkv, dim).
     """
     _need(w, torch.bfloat16, "w", 2)
@@ -1551,7 +1872,7 @@ def skinny_gemm(w: torch.Tensor, tokens: int, *, act: Optional[torch.Tensor] = N
             int(bool(r.get("interleaved", False))), _p(r.get("q_out")), _p(r.get("k_cache")), _p(r.get("v_cache")),
             _p(r.get("positions")), _p(r.get("token_req")), _p(r.get("req_slot")), _p(r.get("block_table")),
             r["block_table"].shape[1] if rope else 0, int(r.get("page_size", 0)), int(r.get("hq", 0)), int(r.get("hkv", 0)),
-            int(r.get("dim", 0)), int(bool(accumulate)), ctypes.c_float(out_mult), _stream())
+            int(r.get("dim", 0)), int(bool(accumulate)), ctypes.c_float(out_mult), GATE_ACTIVATIONS[gate], _stream())
     if (accumulate or out_mult != 1.0) and epilogue != EPI_PLAIN:
         raise KernelError("skinny_gemm: only the plain epilogue adds into its output or multiplies it")
     if kind not in ("auto", "latency", "stream"):
@@ -1632,14 +1953,15 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate
     return out
 
 
-def gemm_tcgen05_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """out (bfloat16 [M, I]) = silu(a @ w[:I]^T) * (a @ w[I:]^T): the product with SwiGLU as its epilogue."""
+def gemm_tcgen05_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: str = "silu") -> torch.Tensor:
+    """out (bfloat16 [M, I]) = act(a @ w[:I]^T) * (a @ w[I:]^T): the product with the gated activation (silu, or the tanh
+    form of gelu) as its epilogue."""
     _need(a, torch.bfloat16, "a", 2); _need(w, torch.bfloat16, "w", 2); _need(out, torch.bfloat16, "out", 2)
     m, k = a.shape
     inter = out.shape[1]
     if w.shape != (2 * inter, k) or out.shape[0] != m:
         raise KernelError(f"gemm swiglu: shapes a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)} disagree")
-    _check(_tcgen05().cisr_gemm_tcgen05_swiglu(_p(a), _p(w), _p(out), m, inter, k, _stream()), "gemm_tcgen05_swiglu")
+    _check(_tcgen05().cisr_gemm_tcgen05_swiglu(_p(a), _p(w), _p(out), m, inter, k, GATE_ACTIVATIONS[gate], _stream()), "gemm_tcgen05_swiglu")
     return out
 
 
@@ -1784,7 +2106,7 @@ _DESCRIBE = {
     "gemm_tcgen05_grouped_gated": lambda a, w, out, tile_group, limit, rows_in_use=None:
         (int(rows_in_use or a.shape[0]), int(w.shape[0]), int(w.shape[1]), int(w.shape[2])),
     "gemm_heads": lambda a, w, out, w_is_nk: (int(a.shape[0]), int(w.shape[0]), int(w.shape[1]), int(w.shape[2])),
-    "swiglu": lambda gate_up, out: (int(out.shape[0]), int(out.shape[1])),
+    "swiglu": lambda gate_up, out, gate="silu": (int(out.shape[0]), int(out.shape[1])),
     "rotary_tables": lambda positions, inv_freq, cos, sin, magnitude=1.0: (int(cos.shape[0]), int(cos.shape[1])),
     "hyper_mix_norm": lambda source, streams, n_streams, **kw:
         (int(streams.shape[0] if kw.get("h") is None else kw["h"].shape[0]), int(n_streams), int(streams.shape[2]), kw.get("y") is not None,
@@ -1808,6 +2130,18 @@ _DESCRIBE = {
     "lightning_recurrence": lambda proj, q_col, k_col, v_col, decay, state, req_slot, q_start, q_len, n_req, o, heads, key_dim, value_dim, **kw:
         (int(proj.shape[0]), int(n_req), int(heads), int(key_dim), int(value_dim), int(kw["chunks"][3]) if kw.get("chunks") else 0),
     "lightning_output": lambda o, *a, **kw: (int(o.shape[0]), int(o.shape[1])),
+    # bytes a launch must move: (rows, hidden, pending, extra, stored, normed)
+    "post_norm": lambda x, **kw: (int(x.shape[0] if kw.get("rows") is None else kw["rows"].numel()), int(x.shape[1]), kw.get("y") is not None,
+                                  kw.get("extra") is not None, kw.get("x_out") is not None, kw.get("h") is not None),
+    "gated_recurrence": lambda q, q_col, k, k_col, v, v_col, la, g, state, req_slot, q_start, q_len, n_req, y, groups, key_dim, **kw:
+        (int(y.shape[0]), int(n_req), int(y.shape[1]), int(groups), int(key_dim), int(y.shape[2]), int(kw["chunks"][3]) if kw.get("chunks") else 0),
+    "short_conv": lambda proj, col, taps_w, *a, **kw: (int(proj.shape[0]), int(taps_w.shape[1]), int(taps_w.shape[0]), kw.get("split") is not None),
+    "exp_gates": lambda proj, i_col, f_col, i_bias, *a, **kw: (int(proj.shape[0]), int(i_bias.shape[0])),
+    "exp_output": lambda y, *a, **kw: (int(y.shape[0]), int(y.shape[1] * y.shape[2])),
+    "ssd_output": lambda y, *a, **kw: (int(y.shape[0]), int(y.shape[1] * y.shape[2]), 0 if kw.get("lead") is None else int(kw["lead"].shape[1])),
+    "rglru_gates": lambda u, w, bias, pre: (int(u.shape[0]), int(w.shape[0]), int(w.shape[2]), int(w.element_size())),
+    "rglru_step": lambda u, w, *a: (int(u.shape[0]), int(w.shape[0]), int(w.shape[2])),
+    "rglru_scan": lambda pre, bias, u, *a, **kw: (int(u.shape[0]), int(u.shape[1])),
     "diff_combine": lambda mixed, gate, gate_col, out, *a: (int(out.shape[0]), int(out.shape[1]), int(mixed.shape[1] * mixed.shape[2])),
     "depth_mix_norm": lambda hist, x, pending, w, n_new, **kw:
         (int(x.shape[0] if kw.get("rows") is None else kw["rows"].numel()), int(n_new), int(x.shape[1]), pending is not None,

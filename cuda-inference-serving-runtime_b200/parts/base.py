@@ -65,6 +65,10 @@ class Part:
         sends to the device inside the step's one metadata copy (`ctx.plan_for(part)` reads it)."""
         return None
 
+    def planning_parts(self) -> list:
+        """The parts whose plans this one uses: itself, or the parts it is made of."""
+        return [self]
+
     def step_plan(self, host):
         """The `engine.batch.StepPlan` for a step described by `host` (`engine.batch.HostBatch`)."""
         raise NotImplementedError

@@ -91,6 +91,9 @@ class PassVectors(Part):
         return [("elementwise.cu", {}, ())]
 
     def add_to(self, stream, index: int) -> None:
-        """stream.x += (pending output, scaled) + row `index`, in one pass; nothing stays pending."""
+        """stream.x += (pending output, scaled) + row `index`, in one pass; nothing stays pending.  A stream that adds vectors
+        in the kernel that reads it next is told the row instead."""
+        if hasattr(stream, "add_vector"):
+            return stream.add_vector(self.rows[index])
         scale = getattr(stream, "pending_scale", None)
         kernels.stream_add(stream.x, stream.take_pending(), scale, self.rows[index])

@@ -1,4 +1,4 @@
-"""SwiGLU feed-forward: down(silu(gate(h)) * up(h)).
+"""SwiGLU feed-forward: down(silu(gate(h)) * up(h)), or with the tanh form of gelu on the gate.
 
 Parity: runtime/model.py:116-119, kernels/execution.cu:7-10.  gate_proj and up_proj
 are stacked into one [2I, H] matrix at load so one product serves both.
@@ -16,7 +16,8 @@ from .linear import as_tensor, linear, linear_to_stream, norm_fusable
 
 @register(FEED_FORWARDS, "swiglu")
 class SwiGLU(FeedForward):
-    """params: hidden_size, intermediate_size; names (local tensor names of gate, up, down)."""
+    """params: hidden_size, intermediate_size; activation of the gate ("silu", the default, or "gelu_tanh"); names (local
+    tensor names of gate, up, down)."""
 
     accepts_pending_norm = True
 
@@ -25,6 +26,9 @@ class SwiGLU(FeedForward):
         self.hidden = int(spec["hidden_size"])
         self.inter = int(spec["intermediate_size"])
         self.names = dict({"gate": "gate_proj.weight", "up": "up_proj.weight", "down": "down_proj.weight"}, **dict(spec.get("names") or {}))
+        self.activation = spec.get("activation", "silu")
+        if self.activation not in kernels.GATE_ACTIVATIONS:
+            raise ValueError(f"unknown gate activation {self.activation!r}")
         self.gate_up = None
         self.down = None
 
@@ -51,16 +55,16 @@ class SwiGLU(FeedForward):
             if norm_fusable(h, tokens, self.gate_up):
                 x_out = h.new_stream_buffer()
                 kernels.skinny_gemm(self.gate_up, tokens, x=h.x, delta=h.delta, norm_w=h.weight, eps=h.eps, x_out=x_out,
-                                    epilogue=kernels.EPI_SWIGLU, out=act)
+                                    epilogue=kernels.EPI_SWIGLU, out=act, gate=self.activation)
                 h.done(x_out)
             else:
-                kernels.skinny_gemm(self.gate_up, tokens, act=as_tensor(h), epilogue=kernels.EPI_SWIGLU, out=act)
+                kernels.skinny_gemm(self.gate_up, tokens, act=as_tensor(h), epilogue=kernels.EPI_SWIGLU, out=act, gate=self.activation)
         else:
             hn = as_tensor(h)
             if kernels.tcgen05_ok(hn, self.gate_up):
-                kernels.gemm_tcgen05_swiglu(hn, self.gate_up, act)      # many tokens: SwiGLU is the product's epilogue
+                kernels.gemm_tcgen05_swiglu(hn, self.gate_up, act, gate=self.activation)      # many tokens: SwiGLU is the product's epilogue
             else:
-                kernels.swiglu(linear(hn, self.gate_up), act)
+                kernels.swiglu(linear(hn, self.gate_up), act, gate=self.activation)
         return linear_to_stream(act, self.down, h0)
 
 

@@ -22,6 +22,21 @@ def linear(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return kernels.gemm(a, w, out)
 
 
+def linear_times(a: torch.Tensor, w: torch.Tensor, mult: float) -> torch.Tensor:
+    """mult * (a . w^T), float [tokens, out]: the factor is the product's epilogue where a kernel has one, else a kernel of
+    its own after the library product."""
+    if mult == 1.0 or a.shape[0] == 0:
+        return linear(a, w)
+    if kernels.skinny_ok(a.shape[0], w) and a.dtype == torch.bfloat16:
+        out = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float32, device=a.device)
+        kernels.skinny_gemm(w, a.shape[0], act=a, epilogue=kernels.EPI_PLAIN, out=out, out_mult=mult)
+        return out
+    if kernels.tcgen05_ok(a, w):
+        out = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float32, device=a.device)
+        return kernels.gemm_tcgen05(a, w, out, out_mult=mult)
+    return kernels.scale_(linear(a, w), mult)
+
+
 def linear_add(a: torch.Tensor, w: torch.Tensor, into: torch.Tensor) -> torch.Tensor:
     """into += a . w^T for a float `into` [tokens, out]: the add is the product's epilogue where a kernel has one (the
     weight-streaming kernels for few tokens, the tcgen05 product for many), else a kernel of its own after the library

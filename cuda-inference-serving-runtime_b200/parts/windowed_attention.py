@@ -4,6 +4,8 @@ window of keys, a sink in the softmax, rotation of part of each head.
 
     q = W_q h (+ b_q), k = W_k h (+ b_k), v = W_v h (+ b_v)        or v = k as projected (no W_v; value_dim = key_dim)
     qk_norm "whole": q <- q / sqrt(mean(q^2) + eps) * w_q with the mean over ALL heads of the token at once; k likewise
+    qk_norm "head": the same head by head, with one weight of a head's size shared by all heads
+    q_temp (coef, every): q <- q * (1 + coef * ln(floor((position + 1) / every) + 1))
     rotation of the first `position.dim` coordinates of each head of q and k
     score = (q . k) * scale over the keys j with 0 <= i - j (< window)
     p_j = exp(s_j) / (sum exp(s) [+ exp(sink)]);  out = W_o [heads of sum_j p_j v_j] (+ b_o)
@@ -32,7 +34,7 @@ HEAD_STEP, HEAD_MAX = 16, 256      # the attention kernels are built per head wi
 @register(MIXERS, "windowed_attention")
 class WindowedAttention(Mixer):
     """params: hidden_size, num_heads, num_kv_heads, key_dim, value_dim, position (PartSpec), scale, window (None or int),
-    sink (None, or the score of the sink), qk_norm (None or "whole"), eps (of that norm), values_from_keys (bool),
+    sink (None, or the score of the sink), qk_norm (None, "whole" or "head"), q_temp (None or (coef, every)), eps (of that norm), values_from_keys (bool),
     bias (the set of projections that have one, among "q", "k", "v", "o"), names."""
 
     graph_safe = True
@@ -49,13 +51,14 @@ class WindowedAttention(Mixer):
         self.window = spec.get("window")
         self.sink = spec.get("sink")
         self.qk_norm = spec.get("qk_norm")
+        self.q_temp = spec.get("q_temp")
         self.eps = float(spec.get("eps", 0.0))
         self.values_from_keys = bool(spec.get("values_from_keys", False))
         self.bias = frozenset(spec.get("bias", ()))
         self.names = {**DEFAULT_NAMES, **dict(spec.get("names") or {})}
         if self.hq % self.hkv:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
-        if self.qk_norm not in (None, "whole"):
+        if self.qk_norm not in (None, "whole", "head"):
             raise ValueError(f"unknown qk_norm {self.qk_norm!r}")
         if self.values_from_keys and (self.value_dim != self.key_dim or "v" in self.bias):
             raise ValueError("values taken from the keys have the keys' width and no projection of their own")
@@ -80,8 +83,9 @@ class WindowedAttention(Mixer):
             if which in self.bias:
                 needs[n[which + "_bias"]] = TensorNeed((size,), role="vector", init_mean=0.0)
         if self.qk_norm:
-            needs[n["q_norm"]] = TensorNeed((nq,), role="vector")
-            needs[n["k_norm"]] = TensorNeed((nk,), role="vector")
+            per_head = self.qk_norm == "head"
+            needs[n["q_norm"]] = TensorNeed((self.key_dim if per_head else nq,), role="vector")
+            needs[n["k_norm"]] = TensorNeed((self.key_dim if per_head else nk,), role="vector")
         return needs
 
     def load(self, tensors):
@@ -123,22 +127,26 @@ class WindowedAttention(Mixer):
     def begin_step(self, ctx) -> None:
         self.position.rotation(ctx)
 
-    def forward(self, h, ctx, cache):
+    def attend(self, proj, ctx, cache) -> torch.Tensor:
+        """From the projection of h (float [tokens, q | k (| v) | columns of other readers]) to the operand of the output
+        projection, [tokens, num_heads * width]."""
         if not cache.write:
             raise NotImplementedError("windowed_attention writes its own keys and values")
         tokens = ctx.n_tokens
         rot = self.position.rotation(ctx)
-        proj = linear(as_tensor(h), self.w_in)                      # float [tokens, q | k (| v)]
         q = torch.empty((tokens, self.hq, self.width), dtype=self.dtype, device=ctx.device)
         kernels.attention_rows(proj, self.k_col, self.v_col, bias=self.in_bias, q_norm=self.q_norm, k_norm=self.k_norm, eps=self.eps,
                                cos=rot.cos if rot else None, sin=rot.sin if rot else None, rot_half=rot.rot_half if rot else 0,
                                interleaved=rot.interleaved if rot else False, q_out=q, k_cache=cache.k, v_cache=cache.v,
                                token_req=ctx.token_req, positions=ctx.positions, req_slot=ctx.req_slot,
                                block_table=cache.block_table, page_size=cache.page_size, hq=self.hq, hkv=self.hkv,
-                               key_dim=self.key_dim, value_dim=self.value_dim)
+                               key_dim=self.key_dim, value_dim=self.value_dim, norm_per_head=self.qk_norm == "head", q_temp=self.q_temp)
         mixed = paged_attention(ctx.plan_for(self), q, cache.k, cache.v, cache, ctx, self.hq, self.hkv, self.scale, self.window,
                                 sink=self.sink)
-        y = linear(mixed.view(tokens, self.hq * self.width), self.o)
+        return mixed.view(tokens, self.hq * self.width)
+
+    def forward(self, h, ctx, cache):
+        y = linear(self.attend(linear(as_tensor(h), self.w_in), ctx, cache), self.o)
         if self.output_bias is not None and not self.bias_taken_by_arrangement:
             kernels.bias_add(y, self.output_bias)
         return y
