@@ -168,7 +168,7 @@ exp_gates_kernel(const float* __restrict__ proj, int stride, int i_col, int f_co
             g[at] = expf(i - m);
             m_out[at] = m;
         }
-        if (threadIdx.x == blockDim.x - 1) carry = m;         // tokens beyond the portion change nothing
+        if (in && (threadIdx.x == blockDim.x - 1 || t == n - 1)) carry = m;      // the very number that the last token's la and g were formed with
         __syncthreads();
         m_before = carry;
     }

@@ -170,12 +170,13 @@ def gated_ff(w: dict, p: str, h: torch.Tensor) -> torch.Tensor:
 MIXERS = {"parallel": parallel, "rglru": rglru, "mlstm": mlstm}
 
 
-def layer(w: dict, cfg: dict, i: int, x: torch.Tensor) -> torch.Tensor:
+def layer(w: dict, cfg: dict, i: int, x: torch.Tensor, taken=lambda h: h) -> torch.Tensor:
+    """`taken`: what a sub-block makes of its normed input before anything else (a rounding, to see what that alone does)."""
     spec, eps, p = cfg["layers"][i], cfg["norm"]["eps"], f"l{i}."
-    y = MIXERS[spec["type"]](w, p + "mix.", spec["mixer"], layer_norm(x, w[p + "norm1"], eps), eps)
+    y = MIXERS[spec["type"]](w, p + "mix.", spec["mixer"], taken(layer_norm(x, w[p + "norm1"], eps)), eps)
     x = x + layer_norm(y, w[p + "norm1b"], eps) * w[p + "ls1"]
     if spec.get("mlp"):
-        y = gated_ff(w, p + "mlp.", layer_norm(x, w[p + "norm2"], eps))
+        y = gated_ff(w, p + "mlp.", taken(layer_norm(x, w[p + "norm2"], eps)))
         x = x + layer_norm(y, w[p + "norm2b"], eps) * w[p + "ls2"]
     return x
 
@@ -192,7 +193,7 @@ def run_order(cfg: dict) -> list:
     return out + [(i, None) for i in range(stop, n)]
 
 
-def streams(cfg: dict, w: dict, tokens) -> list:
+def streams(cfg: dict, w: dict, tokens, taken=lambda h: h) -> list:
     """The residual stream after every layer run."""
     embedded = w["embed"][torch.tensor(list(tokens))] * cfg["embedding"]["scale"]
     x, out = embedded, []
@@ -201,7 +202,7 @@ def streams(cfg: dict, w: dict, tokens) -> list:
             if t > 0:
                 x = x + embedded
             x = x + w["loop.step"][t]
-        x = layer(w, cfg, i, x)
+        x = layer(w, cfg, i, x, taken)
         out.append(x)
     return out
 
@@ -210,9 +211,9 @@ def logits_of(cfg: dict, w: dict, x: torch.Tensor) -> torch.Tensor:
     return layer_norm(x, w["final.norm"], cfg["norm"]["eps"]) @ w["embed"].T
 
 
-def forward(cfg: dict, w: dict, tokens) -> torch.Tensor:
+def forward(cfg: dict, w: dict, tokens, taken=lambda h: h) -> torch.Tensor:
     """Float64 logits [len(tokens), vocab]."""
-    return logits_of(cfg, w, streams(cfg, w, tokens)[-1])
+    return logits_of(cfg, w, streams(cfg, w, tokens, taken)[-1])
 
 
 def generate_greedy(cfg: dict, w: dict, prompt, n: int) -> list:
