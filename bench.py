@@ -27,12 +27,13 @@ every request holding about 4096 tokens of context while it decodes.  Prints ONE
 --workload mixed: the continuous-batching workload (by default the SmolLM2-1.7B sizes, 64 requests with prompts
 of 128 to 2048 tokens, 256 generated tokens each) through the scheduler with graphs on; prints total, prefill
 and decode tokens per second, launch counts, graph statistics and a roofline for the whole run.
---designs SIZES [--design zurolorn|ronolorn|gipozen|vilodra]: Zurolorn (latent attention, routed experts), Ronolorn (windowed
+--designs SIZES [--design zurolorn|ronolorn|gipozen|vilodra|kezunex]: Zurolorn (latent attention, routed experts), Ronolorn (windowed
 attention, gated delta rule, several residual streams), Gipozen (differential attention with convolved projections,
-depth-weighted average of the stream, PolyNorm and routed gated feed-forwards) or Vilodra (lightning attention with a state
-per head, differential attention with rotary positions, windowed latent attention with sinks, gelu experts) beside the
-Llama shape of equal size at the named widths:
-prompt and decode tokens per second of both, and per kind of kernel the device time and the distance from the roofline.
+depth-weighted average of the stream, PolyNorm and routed gated feed-forwards), Vilodra (lightning attention with a state
+per head, differential attention with rotary positions, windowed latent attention with sinks, gelu experts) or Kezunex
+(softmax attention beside a state-space mixer, real-gated linear recurrence, matrix memory; the designs whose kernels are
+most like its own, Ronolorn and Vilodra, stand beside it too) beside the Llama shape of equal size at the named widths:
+prompt and decode tokens per second of each, and per kind of kernel the device time and the distance from the roofline.
 --impl reference: the reference's own stock code on the same decode workload (see reference_arm).
 
 Peaks come from MEASURED_PEAKS.json beside this file when the driver wrote it, else 6.65 TB/s and
@@ -519,6 +520,25 @@ def vilodra_pair(width: int, layers: int, heads: int, ff_active: int, experts: i
     return {"vilodra": vilo, "llama": llama, "zurolorn": zur}
 
 
+def kezunex_pair(width: int, layers: int, heads: int, ff_active: int, experts: int = 0, top: int = 0, vocab: int = 32000):
+    """A Kezunex shape and the Llama shape of equal size beside it: the same width, layers, vocabulary and dense feed-forward in
+    every layer.  Layers in the order pair, recurrent unit, pair, matrix memory; in a pair, half as many query heads of 64 as
+    Llama (an eighth as many key heads) beside a state-space mixer of half the width (heads of 64, states of 128 rows, one
+    group, four taps); recurrent units as wide as the model in parts of 256; matrix memories with keys of 128 and values of 256 per
+    head.  No loop: equal layers run.  Ronolorn and Vilodra, the designs with the like kernels, of the same sizes beside them."""
+    att = {"heads": heads // 2, "kv_heads": max(1, heads // 8), "dim": 64, "vdim": 64, "scale": 0.125, "q_temp": {"coef": 0.1, "every": 1024}}
+    ssm = {"heads": heads // 2, "vdim": width // heads, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    pair = {"left": att, "left_scale": 1.0, "right": ssm, "right_scale": 0.7}
+    unit = {"width": width, "blocks": max(1, width // 256), "conv": 4}
+    memory = {"heads": max(1, width // 256), "dim": 128, "vdim": 256, "gate_cap": 15.0}
+    order = [("parallel", pair), ("rglru", unit), ("parallel", pair), ("mlstm", memory)]
+    keze = {"architecture": "Kezunex", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "max_positions": 8192,
+            "layers": [{"type": order[i % 4][0], "mixer": order[i % 4][1], "mlp": {"kind": "dense", "ff": ff_active}} for i in range(layers)]}
+    others = vilodra_pair(width, layers, heads, ff_active, experts, top, vocab)
+    return {"kezunex": keze, "llama": others["llama"], "ronolorn": ronolorn_pair(width, layers, heads, ff_active, experts, top, vocab)[0],
+            "vilodra": others["vilodra"]}
+
+
 DESIGN_SIZES = {"1024": (1024, 8, 16, 2048, 16, 4), "2048": (2048, 8, 32, 4096, 32, 4), "4096": (4096, 4, 32, 8192, 64, 8)}
 KERNEL_KIND = {   # which kernels of the two designs are alike
     "gemm_tcgen05": "product, many tokens", "gemm_library": "product, many tokens", "gemm_tcgen05_swiglu": "feed-forward product, many tokens",
@@ -532,7 +552,9 @@ KERNEL_KIND = {   # which kernels of the two designs are alike
     "hyper_mix_norm": "norm", "attention_rows": "row kernels", "activation": "row kernels", "delta_prepare": "row kernels",
     "delta_output": "row kernels", "delta_keep": "bookkeeping", "delta_recurrence": "recurrence", "delta_chunks": "recurrence",
     "diff_rows": "row kernels", "diff_combine": "row kernels", "conv_keep": "bookkeeping", "depth_mix_norm": "norm", "polynorm": "row kernels",
-    "gated_clamp": "row kernels", "lightning_recurrence": "recurrence", "lightning_output": "row kernels", "diff_rope_rows": "row kernels"}
+    "gated_clamp": "row kernels", "lightning_recurrence": "recurrence", "lightning_output": "row kernels", "diff_rope_rows": "row kernels",
+    "post_norm": "norm", "gated_recurrence": "recurrence", "short_conv": "row kernels", "exp_gates": "row kernels", "exp_output": "row kernels",
+    "ssd_output": "row kernels", "rglru_gates": "product per part", "rglru_step": "recurrence", "rglru_scan": "recurrence"}
 
 
 def generic_need(name: str, shape: tuple, cache_tokens: int, causal: int):
@@ -601,6 +623,32 @@ def generic_need(name: str, shape: tuple, cache_tokens: int, causal: int):
         # float on the CUDA cores (about four operations per state element and token), which the tensor-core peak does not describe
         tokens, n_req, heads, dk, dv, n_long = shape
         return (n_req * 2 * heads * dk * dv + tokens * heads * (2 * dk + 2 * dv)) * 4, 0.0
+    if name == "gated_recurrence":
+        # the state once in and once out per request, the tokens' operands once in, the read-outs once out; bytes only, as above
+        tokens, n_req, heads, groups, dk, dv, n_long = shape
+        return (n_req * 2 * heads * dk * dv + tokens * (2 * groups * dk + 2 * heads * dv + 2 * heads)) * 4, 0.0
+    if name == "rglru_scan":
+        tokens, width = shape
+        return tokens * width * (4 * 4 + 2), 0.0                  # two gates' sums, u and the output gate in, the operand out
+    if name == "rglru_step":
+        tokens, blocks, block = shape
+        return 2 * blocks * block * block * 2 + tokens * blocks * block * (8 + 8 + 2), 4.0 * tokens * blocks * block * block
+    if name == "rglru_gates":
+        tokens, blocks, block, size = shape
+        return 2 * blocks * block * block * size + tokens * blocks * block * 12, 0.0
+    if name == "post_norm":
+        rows, hidden, pending, extra, stored, normed = shape
+        return rows * hidden * (4 * (1 + pending + extra + stored) + 2 * normed), 0.0
+    if name == "short_conv":
+        tokens, channels, taps, split = shape
+        return tokens * channels * (8 + (6 if split else 0)), 2.0 * tokens * channels * taps
+    if name == "exp_gates":
+        return shape[0] * shape[1] * 20, 0.0
+    if name == "exp_output":
+        return shape[0] * shape[1] * 10, 0.0
+    if name == "ssd_output":
+        tokens, inner, lead = shape
+        return tokens * (inner * 14 + lead * 4), 0.0
     if name == "lightning_output":
         return shape[0] * shape[1] * 10, 0.0
     if name == "diff_rope_rows":
@@ -699,7 +747,7 @@ def design_comparison(args, hbm_gbs: float, burst_tflops: float, peak_source: st
 
     sizes = [s for s in args.designs.split(",") if s]
     batch, context, prompt = args.batch, min(args.context, 2048), PREFILL_TOKENS
-    pair = {"ronolorn": ronolorn_pair, "gipozen": gipozen_pair, "vilodra": vilodra_pair}.get(args.design, design_pair)
+    pair = {"ronolorn": ronolorn_pair, "gipozen": gipozen_pair, "vilodra": vilodra_pair, "kezunex": kezunex_pair}.get(args.design, design_pair)
     line = {"designs": f"{args.design} beside llama at equal size", "dtype": "bf16", "data": "synthetic token ids, seeded random weights",
             "batch": batch, "context": context, "prompt_tokens": prompt, "peaks": peak_source, "sizes": {}}
     sampler = ClockSampler().start()
@@ -963,11 +1011,12 @@ def main() -> int:
     parser.add_argument("--designs", metavar="SIZES", default=None,
                         help="instead of the default workload: Zurolorn beside the Llama shape of equal size, prompt and decode, at "
                              "the named widths (comma-separated, from 1024, 2048, 4096)")
-    parser.add_argument("--design", choices=["zurolorn", "ronolorn", "gipozen", "vilodra"], default="zurolorn",
+    parser.add_argument("--design", choices=["zurolorn", "ronolorn", "gipozen", "vilodra", "kezunex"], default="zurolorn",
                         help="--designs: which design stands beside the Llama shape (ronolorn: windowed attention, gated delta rule, "
                              "four residual streams, dense feed-forward; gipozen: differential attention, depth-weighted average, "
                              "PolyNorm and routed gated feed-forwards; vilodra: lightning attention, differential attention with "
-                             "rotary positions, windowed latent attention with sinks, dense gated and routed gelu feed-forwards)")
+                             "rotary positions, windowed latent attention with sinks, dense gated and routed gelu feed-forwards; "
+                             "kezunex: softmax attention beside a state-space mixer, real-gated linear recurrence, matrix memory)")
     args = parser.parse_args()
     if args.workload == "mixed" and "--preset" not in " ".join(sys.argv):
         args.preset = "smollm2-1.7b"

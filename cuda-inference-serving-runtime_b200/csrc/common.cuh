@@ -58,7 +58,7 @@ __device__ __forceinline__ float warp_max(float v) {
 // gelu in its tanh form, 0.5 z (1 + tanh(u)) with u = sqrt(2 / pi) (z + 0.044715 z^3), written as z / (1 + exp(-2 u)).
 __device__ __forceinline__ float gelu_tanh(float z) {
     const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
-    return z / (1.f + expf(-2.f * u));
+    return __fdividef(z, 1.f + expf(-2.f * u));      // a divisor beyond 2^126 gives 0, which z over it is to float
 }
 
 // Activation of the gate in a gated feed-forward: silu (kind 0) or the tanh form of gelu (kind 1).

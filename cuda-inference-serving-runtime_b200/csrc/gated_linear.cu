@@ -19,8 +19,8 @@
 //           tokens and S0 the state before it:
 //               y_t = exp(L_t) S0^T q_t + sum_{i <= t} exp(L_t - L_i) g_i (q_t . k_i) v_i
 //               S   = exp(L_n) S0 + sum_i exp(L_n - L_i) g_i k_i v_i^T
-//           scores  q_t . k_i per (chunk, group): every head of a group reads them
-//           gains   the last sum of S, for every chunk at once, into a scratch block per (chunk, head)
+//           gains   the last sum of S, for every chunk at once, into a scratch block per (chunk, head); in further CTAs of the
+//                   same launch the scores q_t . k_i per (chunk, group), which every head of a group reads
 //           scan    walks a request's chunks element by element: a block receives the state BEFORE its chunk
 //           reads   the read-outs of every chunk at once: one running product over [q exp(L) | scores with their decays] and [S0 ; v]
 //           Each is a 64 x 64 tile per CTA of 128 threads with 8 x 4 results per thread, float on the CUDA cores.
@@ -224,17 +224,10 @@ __device__ __forceinline__ void stage_decays(const Args& a, int h, int token0, i
     }
 }
 
+// q_t . k_i of one chunk and group (n tokens from row token0 on), every pair of tokens
 template <bool VEC>
-__global__ void __launch_bounds__(THREADS)
-gated_scores_kernel(const Args a) {
-    extern __shared__ __align__(16) float smem[];
-    float* Q = smem;
-    float* K = Q + CHUNK * LDT;
-    pdl_trigger();
-    const int chunk = blockIdx.x, grp = blockIdx.y, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    const int r = a.chunk_req[chunk], t0 = a.chunk_t0[chunk], n = min(CHUNK, a.q_len[r] - t0);
-    const size_t token0 = (size_t)(a.q_start[r] + t0);
-    pdl_wait();
+__device__ __forceinline__ void chunk_scores(const Args& a, int chunk, int grp, int n, size_t token0, float* Q, float* K) {
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     float acc[8][4] = {};
     for (int n0 = 0; n0 < a.N; n0 += CHUNK) {
         const int nc = min(CHUNK, a.N - n0);
@@ -244,18 +237,18 @@ gated_scores_kernel(const Args a) {
         __syncthreads();
         const int k4s = (nc + 3) >> 2;
         for (int k4 = 0; k4 < k4s; ++k4) {
-            float4 q[8], k[4];
-#pragma unroll
-            for (int x = 0; x < 8; ++x) q[x] = *reinterpret_cast<const float4*>(Q + (ty + 8 * x) * LDT + 4 * k4);
+            float4 k[4];
 #pragma unroll
             for (int y = 0; y < 4; ++y) k[y] = *reinterpret_cast<const float4*>(K + (tx + 16 * y) * LDT + 4 * k4);
 #pragma unroll
-            for (int x = 0; x < 8; ++x)
+            for (int x = 0; x < 8; ++x) {
+                const float4 q = *reinterpret_cast<const float4*>(Q + (ty + 8 * x) * LDT + 4 * k4);
 #pragma unroll
                 for (int y = 0; y < 4; ++y) {
-                    acc[x][y] = fmaf(q[x].x, k[y].x, acc[x][y]); acc[x][y] = fmaf(q[x].y, k[y].y, acc[x][y]);
-                    acc[x][y] = fmaf(q[x].z, k[y].z, acc[x][y]); acc[x][y] = fmaf(q[x].w, k[y].w, acc[x][y]);
+                    acc[x][y] = fmaf(q.x, k[y].x, acc[x][y]); acc[x][y] = fmaf(q.y, k[y].y, acc[x][y]);
+                    acc[x][y] = fmaf(q.z, k[y].z, acc[x][y]); acc[x][y] = fmaf(q.w, k[y].w, acc[x][y]);
                 }
+            }
         }
     }
     float* out = a.scores + ((size_t)chunk * a.groups + grp) * CHUNK * CHUNK;
@@ -265,8 +258,9 @@ gated_scores_kernel(const Args a) {
         for (int y = 0; y < 4; ++y) out[(ty + 8 * x) * CHUNK + tx + 16 * y] = acc[x][y];
 }
 
+// grid (chunk, head, tiles of [N, dv] + 1): the last z makes the scores of the chunk's groups, in the CTAs of the first heads
 template <bool VEC, bool NORM>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS, 5)
 gated_gains_kernel(const Args a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ double L[CHUNK];
@@ -275,6 +269,7 @@ gated_gains_kernel(const Args a) {
     float* V = K + CHUNK * LDT;
     pdl_trigger();
     const int chunk = blockIdx.x, h = blockIdx.y, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const bool scores = blockIdx.z == gridDim.z - 1;
     const int row_tiles = (a.N + CHUNK - 1) / CHUNK;
     const int n0 = ((int)blockIdx.z % row_tiles) * CHUNK, c0 = ((int)blockIdx.z / row_tiles) * CHUNK;
     const int grp = h / (a.heads / a.groups);
@@ -282,6 +277,10 @@ gated_gains_kernel(const Args a) {
     const int token0 = a.q_start[r] + t0;
     const int nr = min(CHUNK, a.N - n0), nc = min(CHUNK, a.dv - c0);
     pdl_wait();
+    if (scores) {
+        if (h < a.groups) chunk_scores<VEC>(a, chunk, h, n, (size_t)token0, K, V);
+        return;
+    }
     stage_decays(a, h, token0, n, L, w);
     stage<VEC>(K, a.k + (size_t)token0 * a.k_stride + grp * a.N + n0, a.k_stride, n, nr);
     stage<VEC>(V, a.v + (size_t)token0 * a.v_stride + h * a.dv + c0, a.v_stride, n, nc);
@@ -348,26 +347,39 @@ gated_scan_kernel(const Args a) {
     const size_t step = (size_t)a.heads * per_head;
     float* block = a.blocks + ((size_t)chunk0 * a.heads + h) * per_head + e;
     const float* decay = a.chunk_decay + (size_t)chunk0 * a.heads + h;
-    constexpr int AHEAD = VEC == 1 ? 8 : 4;               // gains requested together: the walk itself is one multiply-add per chunk
-    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        float gain[AHEAD][VEC], f[AHEAD];
+    // the walk itself is one multiply-add per chunk: it goes as fast as the gains arrive, so AHEAD of them are asked for
+    // together, and the next ones before the ones at hand are used
+    constexpr int AHEAD = 8;
+    float gain[AHEAD][VEC], f[AHEAD];
+    const auto fetch = [&](int c0) {
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
             const bool in = c0 + u < chunks;
             f[u] = in ? decay[(size_t)(c0 + u) * a.heads] : 0.f;
-            if (VEC == 4) {
-                const float4 x = in ? *reinterpret_cast<const float4*>(block + (size_t)(c0 + u) * step) : make_float4(0.f, 0.f, 0.f, 0.f);
-                gain[u][0] = x.x; gain[u][1 % VEC] = x.y; gain[u][2 % VEC] = x.z; gain[u][3 % VEC] = x.w;
+            if (VEC == 2) {
+                const float2 x = in ? *reinterpret_cast<const float2*>(block + (size_t)(c0 + u) * step) : make_float2(0.f, 0.f);
+                gain[u][0] = x.x; gain[u][1 % VEC] = x.y;
             } else gain[u][0] = in ? block[(size_t)(c0 + u) * step] : 0.f;
         }
+    };
+    fetch(0);
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        float now[AHEAD][VEC], fn[AHEAD];
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u) {
+            fn[u] = f[u];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) now[u][j] = gain[u][j];
+        }
+        if (c0 + AHEAD < chunks) fetch(c0 + AHEAD);
 #pragma unroll
         for (int u = 0; u < AHEAD; ++u) {
             if (c0 + u < chunks) {
                 float* at = block + (size_t)(c0 + u) * step;
-                if (VEC == 4) *reinterpret_cast<float4*>(at) = make_float4(S[0], S[1 % VEC], S[2 % VEC], S[3 % VEC]);
+                if (VEC == 2) *reinterpret_cast<float2*>(at) = make_float2(S[0], S[1 % VEC]);
                 else at[0] = S[0];
 #pragma unroll
-                for (int j = 0; j < VEC; ++j) S[j] = fmaf(f[u], S[j], gain[u][j]);
+                for (int j = 0; j < VEC; ++j) S[j] = fmaf(fn[u], S[j], now[u][j]);
             }
         }
     }
@@ -378,24 +390,24 @@ gated_scan_kernel(const Args a) {
 // acc[x][y] += sum_k A[ty + 8 x][k] B[k][4 tx + y] over the first 4 * k4s rows of B
 __device__ __forceinline__ void tile_product(const float* A, const float* B, int tx, int ty, int k4s, float (&acc)[8][4]) {
     for (int k4 = 0; k4 < k4s; ++k4) {
-        float4 av[8];
+        float4 b[4];
 #pragma unroll
-        for (int x = 0; x < 8; ++x) av[x] = *reinterpret_cast<const float4*>(A + (ty + 8 * x) * LDT + 4 * k4);
+        for (int kk = 0; kk < 4; ++kk) b[kk] = *reinterpret_cast<const float4*>(B + (4 * k4 + kk) * LDT + 4 * tx);
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
-            const float4 b = *reinterpret_cast<const float4*>(B + (4 * k4 + kk) * LDT + 4 * tx);
+        for (int x = 0; x < 8; ++x) {
+            const float4 av = *reinterpret_cast<const float4*>(A + (ty + 8 * x) * LDT + 4 * k4);
+            const float f[4] = {av.x, av.y, av.z, av.w};
 #pragma unroll
-            for (int x = 0; x < 8; ++x) {
-                const float f = kk == 0 ? av[x].x : kk == 1 ? av[x].y : kk == 2 ? av[x].z : av[x].w;
-                acc[x][0] = fmaf(f, b.x, acc[x][0]); acc[x][1] = fmaf(f, b.y, acc[x][1]);
-                acc[x][2] = fmaf(f, b.z, acc[x][2]); acc[x][3] = fmaf(f, b.w, acc[x][3]);
+            for (int kk = 0; kk < 4; ++kk) {
+                acc[x][0] = fmaf(f[kk], b[kk].x, acc[x][0]); acc[x][1] = fmaf(f[kk], b[kk].y, acc[x][1]);
+                acc[x][2] = fmaf(f[kk], b[kk].z, acc[x][2]); acc[x][3] = fmaf(f[kk], b[kk].w, acc[x][3]);
             }
         }
     }
 }
 
 template <bool VEC, bool NORM>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS, 5)
 gated_reads_kernel(const Args a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ double L[CHUNK];
@@ -494,14 +506,19 @@ template <bool VEC, bool NORM>
 int chunks(const Args& a, int n_req, int n_chunks, cudaStream_t s) {
     const size_t smem = sizeof(float) * 2 * CHUNK * LDT;       // 34 KB: within the default limit
     const int row_tiles = (a.N + CHUNK - 1) / CHUNK, col_tiles = (a.dv + CHUNK - 1) / CHUNK;
-    int st = launch_kernel(gated_scores_kernel<VEC>, dim3(n_chunks, a.groups), dim3(THREADS), smem, s, g_pdl, a);
-    if (st) return st;
-    st = launch_kernel(gated_gains_kernel<VEC, NORM>, dim3(n_chunks, a.heads, row_tiles * col_tiles), dim3(THREADS), smem, s, g_pdl, a);
+    static bool configured = false;
+    if (!configured) {       // five CTAs per SM want more shared memory than the default split gives
+        cudaError_t e = cudaFuncSetAttribute(gated_gains_kernel<VEC, NORM>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_reads_kernel<VEC, NORM>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    int st = launch_kernel(gated_gains_kernel<VEC, NORM>, dim3(n_chunks, a.heads, row_tiles * col_tiles + 1), dim3(THREADS), smem, s, g_pdl, a);
     if (st) return st;
     const int elements = a.N * a.dv + (NORM ? a.N : 0);
-    // four elements per thread where every block and every state row begins on 16 bytes and no run straddles matrix and normaliser
-    const bool quads = VEC && a.N % 4 == 0 && a.state_stride % 4 == 0 && !((uintptr_t)a.state & 15);
-    if (quads) st = launch_kernel(gated_scan_kernel<4, NORM>, dim3(n_req, a.heads, (elements / 4 + 255) / 256), dim3(256), 0, s, g_pdl, a);
+    // two elements per thread where every block and every state row begins on 8 bytes and no pair straddles matrix and normaliser
+    const bool pairs = VEC && a.state_stride % 2 == 0 && !((uintptr_t)a.state & 7);
+    if (pairs) st = launch_kernel(gated_scan_kernel<2, NORM>, dim3(n_req, a.heads, (elements / 2 + 255) / 256), dim3(256), 0, s, g_pdl, a);
     else st = launch_kernel(gated_scan_kernel<1, NORM>, dim3(n_req, a.heads, (elements + 255) / 256), dim3(256), 0, s, g_pdl, a);
     if (st) return st;
     return launch_kernel(gated_reads_kernel<VEC, NORM>, dim3(n_chunks, a.heads, col_tiles), dim3(THREADS), smem, s, g_pdl, a);

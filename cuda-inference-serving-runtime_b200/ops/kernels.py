@@ -1130,7 +1130,7 @@ def gated_recurrence(q: torch.Tensor, q_col: int, k: torch.Tensor, k_col: int, v
         at(q, q_col), q.shape[1], at(k, k_col), k.shape[1], at(v, v_col), v.shape[1], _p(la), _p(g), _p(state), ctypes.c_longlong(state.shape[1]),
         _p(req_slot), _p(q_start), _p(q_len), _p(y), _p(yn), ctypes.c_float(q_scale), heads, groups, key_dim, dv, n_req,
         int(least if n_chunks else 0), int(n_chunks), int(n_short), _p(chunk_req), _p(chunk_t0), _p(req_chunk0), _p(scores), _p(blocks),
-        _p(decays), _stream()), "gated_recurrence", own=(4 if n_chunks else 0) + (1 if not n_chunks or n_short else 0))
+        _p(decays), _stream()), "gated_recurrence", own=(3 if n_chunks else 0) + (1 if not n_chunks or n_short else 0))
     return y
 
 
