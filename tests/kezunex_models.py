@@ -64,7 +64,7 @@ KB = model(263, 128, [
     layer(mlstm(2, 72, 136, cap=15.0), 64),
     layer(parallel(left(2, 2, 32, 128, 0.3), right(2, 80, 64, parts=2), 0.5, 1.0)),
     layer(rglru(192, 4, conv=3)),
-], eps=1e-6, scale=2.0, loop=(0, 3, 3))
+], eps=1e-6, scale=2.0, loop=(0, 2, 4))
 
 # one head, one block, one tap, no loop, scales of 1, a left side that does not count
 KC = model(97, 52, [
