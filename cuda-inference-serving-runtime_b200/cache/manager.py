@@ -9,7 +9,9 @@ passed it (pages that hold the first `keep_first` keys of such a use stay); entr
 fixed-size state get a tensor [slots, ...] each.  A page id means the same page in every
 entry of its group, so one allocation serves all of them.  A paged entry may hold a small
 state besides its pages (`side_states`: the kept inputs of a convolution, say): always its
-own, also where it reads another entry's pages.
+own, also where it reads another entry's pages.  What a model keeps per request ahead of its
+run entries (the newest token, for an embedding that looks at pairs) is a side state behind
+the last entry's.
 
 Every live request holds one slot.  The slot indexes the request's row in each
 group's block table on the device and its row in every state tensor.  Block tables
@@ -102,7 +104,8 @@ class CacheManager:
     `uses[i]` is the `CacheUse` of run entry i, or the index of the earlier entry whose
     cache entry i reads.  `n_pages` pages of `page_size` tokens are given to each page
     group.  `side_states[i]`, where given, is a `CacheUse("state", ...)` that run entry i holds besides
-    its pages (or besides the pages it reads).  With `device=None` only the host bookkeeping exists
+    its pages (or besides the pages it reads); places behind the last run entry are states that belong to no
+    entry (`side_state` gives them).  With `device=None` only the host bookkeeping exists
     (tests of the allocator).
     """
 
@@ -313,12 +316,15 @@ class CacheManager:
         if kind == "pages":
             g = self.page_groups[gi]
             e = g.entry_slot[source]
-            side = self.entry_side.get(entry)
-            state = None if side is None else self.state_groups[side[0]].storage[side[1]]
             return PagedBinding(g.storage[e, 0], g.storage[e, g.use.planes - 1], g.device_table, g.page_size,
-                                write=reads_from is None, window=g.use.window, keep_first=g.use.keep_first, state=state)
+                                write=reads_from is None, window=g.use.window, keep_first=g.use.keep_first, state=self.side_state(entry))
         g = self.state_groups[gi]
         return StateBinding(g.storage[g.entry_slot[source]])
+
+    def side_state(self, place: int) -> Optional[torch.Tensor]:
+        """The side state [slots, ...] asked for at `place` of `side_states`, or None."""
+        side = self.entry_side.get(place)
+        return None if side is None else self.state_groups[side[0]].storage[side[1]]
 
     # ---------------------------------------------------------------- checks and reports
     def check(self) -> None:

@@ -8,8 +8,9 @@ from .ronolorn import RonolornConfig    # registers Ronolorn
 from .gipozen import GipozenConfig      # registers Gipozen
 from .vilodra import VilodraConfig      # registers Vilodra
 from .kezunex import KezunexConfig      # registers Kezunex
+from .tekezen import TekezenConfig      # registers Tekezen
 from .presets import preset, preset_dict, preset_names
 
-__all__ = ["CacheUse", "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "LlamaConfig", "ZurolornConfig", "RonolornConfig", "GipozenConfig", "VilodraConfig", "KezunexConfig",
+__all__ = ["CacheUse", "ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "RunEntry", "LlamaConfig", "ZurolornConfig", "RonolornConfig", "GipozenConfig", "VilodraConfig", "KezunexConfig", "TekezenConfig",
            "ARCHITECTURES", "Architecture", "architecture_for", "register_architecture",
            "preset", "preset_dict", "preset_names"]

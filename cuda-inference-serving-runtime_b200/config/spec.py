@@ -26,7 +26,8 @@ class PartSpec:
 @dataclass(frozen=True)
 class LayerSpec:
     """One layer: a mixer and a feed-forward, each with its norm, and how they are arranged.  A layer without a
-    feed-forward has `feed_forward` and `feed_forward_norm` None (arrangements that allow it say so).  `extras` are
+    feed-forward has `feed_forward` and `feed_forward_norm` None, one whose sub-blocks read the stream itself has the norms None
+    (arrangements that allow it say so).  `extras` are
     further parts of the arrangement by slot name (per-channel scales of the two outputs, for one).
 
     `names` maps the four slots to the sub-prefix their tensors carry in the
@@ -34,7 +35,7 @@ class LayerSpec:
     """
     prefix: str
     mixer: PartSpec
-    mixer_norm: PartSpec
+    mixer_norm: Optional[PartSpec]
     feed_forward: Optional[PartSpec]
     feed_forward_norm: Optional[PartSpec]
     arrangement: str = "pre_norm"

@@ -1,6 +1,6 @@
 // Causal grouped-query attention over the paged cache, in float arithmetic.
 //
-// Compiled once per (HEAD_DIM, STORAGE_BF16): HEAD_DIM any multiple of 16 up to 256;
+// Compiled once per (HEAD_DIM, STORAGE_BF16): HEAD_DIM any multiple of 16 up to 512;
 // STORAGE_BF16=0 reads float queries and a float cache (the true 32-bit path),
 // STORAGE_BF16=1 reads bfloat16 queries and a bfloat16 cache.  Scores, softmax
 // statistics and the value sum are float in both.
@@ -20,13 +20,16 @@
 //
 // Visibility: query i sees key j when j <= i and (window <= 0 or i - j < window or j < keep_first): a window of the
 // latest keys, and optionally the sequence's first `keep_first` keys kept in sight whatever the distance.
+//
+// With -DSOFTCAP=1 a score becomes cap tanh(score / cap) before the softmax (`softcap`; ignored otherwise).
 #include "common.cuh"
+#include "softcap.cuh"
 
 #ifndef HEAD_DIM
-#error "compile with -DHEAD_DIM=<multiple of 16, at most 256>"
+#error "compile with -DHEAD_DIM=<multiple of 16, at most 512>"
 #endif
-#if (HEAD_DIM % 16) || (HEAD_DIM > 256) || (HEAD_DIM < 16)
-#error "HEAD_DIM must be a multiple of 16 between 16 and 256"
+#if (HEAD_DIM % 16) || (HEAD_DIM > 512) || (HEAD_DIM < 16)
+#error "HEAD_DIM must be a multiple of 16 between 16 and 512"
 #endif
 #ifndef STORAGE_BF16
 #define STORAGE_BF16 0
@@ -57,7 +60,7 @@ __device__ __forceinline__ void load_vec(const st_t* p, float* out) {
 
 // ------------------------------------------------------------------ prefill
 constexpr int BM = 64;
-constexpr int BN = (D <= 128) ? 64 : 32;
+constexpr int BN = (D <= 128) ? 64 : (D <= 256) ? 32 : 16;
 constexpr int NJ = BN / 16;  // score columns per thread
 constexpr int ND = D / 16;   // output columns per thread
 constexpr int QS = BM + 4, KS = BN + 4, PS = BM + 4;
@@ -69,8 +72,8 @@ attn_prefill_kernel(const st_t* __restrict__ q, st_t* __restrict__ out, const st
                     const st_t* __restrict__ v_cache, const int* __restrict__ req_slot,
                     const int* __restrict__ block_table, int table_width, const int* __restrict__ tile_req, const int* __restrict__ tile_q0,
                     const int* __restrict__ q_start, const int* __restrict__ q_len,
-                    const int* __restrict__ ctx_len, int hq, int hkv, int page_size, float scale, int window, int keep_first, float sink,
-                    const float* __restrict__ sink_heads) {
+                    const int* __restrict__ ctx_len, int hq, int hkv, int page_size, float scale, float softcap, int window, int keep_first,
+                    float sink, const float* __restrict__ sink_heads) {
     CISR_TRACE_SCOPE(TRACE_ATTN_SIMT);
     extern __shared__ __align__(16) float smem[];
     float* Qs = smem;             // [D][QS]   transposed, pre-scaled
@@ -147,10 +150,12 @@ attn_prefill_kernel(const st_t* __restrict__ q, st_t* __restrict__ out, const st
             float kk[NJ];
             if (NJ == 4) {
                 const float4 k4 = *reinterpret_cast<const float4*>(Ks + d * KS + tx * 4);
-                kk[0] = k4.x; kk[1] = k4.y; kk[NJ - 2] = k4.z; kk[NJ - 1] = k4.w;
-            } else {
+                kk[0] = k4.x; kk[1 % NJ] = k4.y; kk[2 % NJ] = k4.z; kk[NJ - 1] = k4.w;
+            } else if (NJ == 2) {
                 const float2 k2 = *reinterpret_cast<const float2*>(Ks + d * KS + tx * 2);
-                kk[0] = k2.x; kk[1] = k2.y;
+                kk[0] = k2.x; kk[NJ - 1] = k2.y;
+            } else {
+                kk[0] = Ks[d * KS + tx];
             }
             const float qq[4] = {qv.x, qv.y, qv.z, qv.w};
 #pragma unroll
@@ -169,6 +174,7 @@ attn_prefill_kernel(const st_t* __restrict__ q, st_t* __restrict__ out, const st
             for (int j = 0; j < NJ; ++j) {
                 const int kpos = k0 + tx * NJ + j;
                 const bool ok = (r < rows) && (kpos <= qpos) && (window <= 0 || kpos + window > qpos || kpos < keep_first);
+                if (SOFTCAP) s[i][j] = softcap * tanhf(s[i][j] / softcap);
                 s[i][j] = ok ? s[i][j] : -INFINITY;
                 tile_max = fmaxf(tile_max, s[i][j]);
             }
@@ -236,7 +242,7 @@ __global__ void __launch_bounds__(DEC_THREADS)
 attn_decode_kernel(const st_t* __restrict__ q, const st_t* __restrict__ k_cache, const st_t* __restrict__ v_cache,
                    const int* __restrict__ req_slot, const int* __restrict__ block_table, int table_width, const int* __restrict__ dec_req,
                    const int* __restrict__ q_start, const int* __restrict__ ctx_len, float* __restrict__ partial,
-                   float* __restrict__ stats, int hq, int hkv, int page_size, float scale, int window, int keep_first,
+                   float* __restrict__ stats, int hq, int hkv, int page_size, float scale, float softcap, int window, int keep_first,
                    int split_size, int n_splits) {
     CISR_TRACE_SCOPE(TRACE_ATTN_SIMT);
     extern __shared__ __align__(16) float smem[];
@@ -311,6 +317,7 @@ attn_decode_kernel(const st_t* __restrict__ q, const st_t* __restrict__ k_cache,
                 acc = fmaf(a.z, b.z, acc); acc = fmaf(a.w, b.w, acc);
             }
             const int kpos = k0 + t;
+            if (SOFTCAP) acc = softcap * tanhf(acc / softcap);
             ps[g * TK + t] = (kpos < hi && !in_gap(run, kpos)) ? acc : -INFINITY;
         }
         __syncthreads();
@@ -399,10 +406,10 @@ CISR_EXPORT int cisr_attn_prefill_tile() { return BM; }
 CISR_EXPORT int cisr_attn_prefill(const void* q, void* out, const void* k_cache, const void* v_cache,
                                   const int* req_slot, const int* block_table, int table_width, const int* tile_req, const int* tile_q0,
                                   int n_tiles, const int* q_start, const int* q_len, const int* ctx_len, int hq,
-                                  int hkv, int page_size, float scale, int window, int keep_first, float sink, const float* sink_heads,
-                                  void* stream) {
+                                  int hkv, int page_size, float scale, float softcap, int window, int keep_first, float sink,
+                                  const float* sink_heads, void* stream) {
     if (n_tiles <= 0) return 0;
-    if (hq % hkv) return -2;
+    if (hq % hkv || (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f)) return -2;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PREFILL_SMEM);
@@ -411,7 +418,7 @@ CISR_EXPORT int cisr_attn_prefill(const void* q, void* out, const void* k_cache,
     }
     attn_prefill_kernel<<<dim3(n_tiles, hq), PREFILL_THREADS, PREFILL_SMEM, (cudaStream_t)stream>>>(
         (const st_t*)q, (st_t*)out, (const st_t*)k_cache, (const st_t*)v_cache, req_slot, block_table, table_width, tile_req,
-        tile_q0, q_start, q_len, ctx_len, hq, hkv, page_size, scale, window, keep_first, sink, sink_heads);
+        tile_q0, q_start, q_len, ctx_len, hq, hkv, page_size, scale, softcap, window, keep_first, sink, sink_heads);
     return launch_status();
 }
 
@@ -419,10 +426,10 @@ CISR_EXPORT int cisr_attn_prefill(const void* q, void* out, const void* k_cache,
 CISR_EXPORT int cisr_attn_decode(const void* q, void* out, const void* k_cache, const void* v_cache,
                                  const int* req_slot, const int* block_table, int table_width, const int* dec_req, int n_dec,
                                  const int* q_start, const int* ctx_len, float* partial, float* stats, int hq,
-                                 int hkv, int page_size, float scale, int window, int keep_first, int split_size, int n_splits,
+                                 int hkv, int page_size, float scale, float softcap, int window, int keep_first, int split_size, int n_splits,
                                  float sink, const float* sink_heads, void* stream) {
     if (n_dec <= 0) return 0;
-    if (hq % hkv || split_size <= 0 || n_splits <= 0) return -2;
+    if (hq % hkv || split_size <= 0 || n_splits <= 0 || (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f)) return -2;
     const size_t smem = decode_smem_floats(hq / hkv) * sizeof(float);
     if (smem > 220 * 1024) return -3;
     static size_t configured = 48 * 1024;
@@ -434,7 +441,7 @@ CISR_EXPORT int cisr_attn_decode(const void* q, void* out, const void* k_cache, 
     cudaStream_t s = (cudaStream_t)stream;
     attn_decode_kernel<<<dim3(n_dec, hkv, n_splits), DEC_THREADS, smem, s>>>(
         (const st_t*)q, (const st_t*)k_cache, (const st_t*)v_cache, req_slot, block_table, table_width, dec_req, q_start,
-        ctx_len, partial, stats, hq, hkv, page_size, scale, window, keep_first, split_size, n_splits);
+        ctx_len, partial, stats, hq, hkv, page_size, scale, softcap, window, keep_first, split_size, n_splits);
     int status = launch_status();
     if (status) return status;
     attn_merge_kernel<<<dim3(n_dec, hq), D < 128 ? 64 : 128, 0, s>>>(partial, stats, (st_t*)out, dec_req, q_start, hq, n_splits, sink, sink_heads);

@@ -15,8 +15,10 @@
 //   attn_merge   : log-sum-exp merge of the key ranges in a fixed order (kernels/ops.cu:72-86).
 //
 // Scores are scaled by scale * log2(e) in float after the product and exponentials are base 2.
+// With -DSOFTCAP=1 a score becomes cap tanh(score / cap) before the softmax (`softcap`; ignored otherwise).
 // Cache layout: [pages, kv_heads, page_size, HEAD_DIM].
 #include "common.cuh"
+#include "softcap.cuh"
 
 #ifndef HEAD_DIM
 #error "compile with -DHEAD_DIM=<multiple of 16, at most 128>"
@@ -120,8 +122,8 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, cons
                         const bf16* __restrict__ v_cache, const int* __restrict__ req_slot,
                         const int* __restrict__ block_table, int table_width, const int* __restrict__ tile_req,
                         const int* __restrict__ tile_q0, const int* __restrict__ q_start, const int* __restrict__ q_len,
-                        const int* __restrict__ ctx_len, int hq, int hkv, int page_size, float scale, int window, int keep_first, float sink_all,
-                        const float* __restrict__ sink_heads) {
+                        const int* __restrict__ ctx_len, int hq, int hkv, int page_size, float scale, float softcap, int window, int keep_first,
+                        float sink_all, const float* __restrict__ sink_heads) {
     CISR_TRACE_SCOPE(TRACE_ATTN_PREFILL);
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);   // [BM][LDS]
@@ -180,7 +182,7 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, cons
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < ND; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
-    const float scale2 = scale * LOG2E;
+    const float scale2 = SOFTCAP ? 1.f : scale * LOG2E;      // bent scores come in base-2 units
 
     bf16* gbuf = pipe + (size_t)group * NB * 2 * BN * LDS;      // this group's [K tile | V tile] buffers
     if (group < n_tiles) load_tile(gbuf, group);
@@ -212,6 +214,14 @@ attn_prefill_mma_kernel(const bf16* __restrict__ q, bf16* __restrict__ out, cons
             }
         }
 
+        if (SOFTCAP) {
+            const Bend bend(scale, softcap);
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] = bend(s[nt][e]);
+            }
+        }
         // Mask only where a tile can be cut by the causal edge, the window's edge or the tile's row count; most
         // tiles of a long prompt lie wholly inside and skip the per-element test.
         const int warp_row0 = warp * 16;
@@ -350,6 +360,19 @@ constexpr size_t DEC_MERGE_BYTES = sizeof(float) * (size_t)(4 * 16 * (D + 2));
 constexpr size_t DEC_PIPE_BYTES = STAGES * DEC_TILE_BYTES > DEC_MERGE_BYTES ? STAGES * DEC_TILE_BYTES : DEC_MERGE_BYTES;
 constexpr size_t DEC_SMEM = ((sizeof(bf16) * (size_t)(16 * LDS) + DEC_PIPE_BYTES + 15) / 16) * 16;
 
+// A raw product of query and key in base-2 units of the score, bent where the build asks for it.
+struct ScoreUnits {
+#if SOFTCAP
+    Bend bend;
+    __device__ __forceinline__ ScoreUnits(float scale, float softcap) : bend(scale, softcap) {}
+    __device__ __forceinline__ float operator()(float raw) const { return bend(raw); }
+#else
+    float scale2;
+    __device__ __forceinline__ ScoreUnits(float scale, float) : scale2(scale * LOG2E) {}
+    __device__ __forceinline__ float operator()(float raw) const { return raw * scale2; }
+#endif
+};
+
 // Where 16-byte chunk `chunk` of key row `row` of a tile gathered by cp.async lies: rows LDS elements apart.
 struct PaddedTile {
     const bf16* k; const bf16* v;
@@ -360,7 +383,7 @@ struct PaddedTile {
 // k0 is the position of the slab's first key; keys outside the run [lo, hi) and keys of its gap are masked.
 template <typename Tile>
 __device__ __forceinline__ void decode_slab(const Tile& tile, const uint32_t (&qf)[KD][4], float (&o)[ND][4], float (&m_run)[2],
-                                            float (&l_run)[2], int k0, const KeyRun& run, float scale2, int warp, int lane) {
+                                            float (&l_run)[2], int k0, const KeyRun& run, const ScoreUnits& units, int warp, int lane) {
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
     for (int kk = 0; kk < KD; ++kk) {
@@ -375,7 +398,7 @@ __device__ __forceinline__ void decode_slab(const Tile& tile, const uint32_t (&q
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int kpos = k0 + nt * 8 + 2 * (lane & 3) + (e & 1);
-            const float v = (kpos < run.hi && kpos >= run.lo && !in_gap(run, kpos)) ? s[nt][e] * scale2 : -INFINITY;
+            const float v = (kpos < run.hi && kpos >= run.lo && !in_gap(run, kpos)) ? units(s[nt][e]) : -INFINITY;
             s[nt][e] = v;
             tile_max[e >> 1] = fmaxf(tile_max[e >> 1], v);
         }
@@ -467,7 +490,7 @@ attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_ca
                        const int* __restrict__ req_slot, const int* __restrict__ block_table, int table_width,
                        const int* __restrict__ dec_req, const int* __restrict__ q_start, const int* __restrict__ ctx_len,
                        float* __restrict__ partial, float* __restrict__ stats, int hq, int hkv, int page_size,
-                       float scale, int window, int keep_first, int split_size, int n_splits, int row0) {
+                       float scale, float softcap, int window, int keep_first, int split_size, int n_splits, int row0) {
     CISR_TRACE_SCOPE(TRACE_ATTN_DECODE_GATHER);
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);                    // [16][LDS]
@@ -540,7 +563,7 @@ attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_ca
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
 #pragma unroll
     for (int i = 0; i < ND; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
-    const float scale2 = scale * LOG2E;
+    const ScoreUnits units(scale, softcap);
 
     for (int t = 0; t < n_tiles; ++t) {
         if (t == 0 && early) cp_async_wait<0>();       // the early tiles and the query, all issued long ago
@@ -560,7 +583,7 @@ attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_ca
                 ldmatrix_x4(qf[kk], Qs + ((lane & 7) + 8 * ((lane >> 3) & 1)) * LDS + kk * 16 + 8 * (lane >> 4));
         }
         const bf16* Kt = pipe + (t % STAGES) * 2 * BN * LDS;
-        decode_slab(PaddedTile{Kt, Kt + BN * LDS}, qf, o, m_run, l_run, lo + t * BN + warp * 16, run, scale2, warp, lane);
+        decode_slab(PaddedTile{Kt, Kt + BN * LDS}, qf, o, m_run, l_run, lo + t * BN + warp * 16, run, units, warp, lane);
     }
     cp_async_wait<0>();
     __syncthreads();          // every warp is done with the pipeline buffers: they become the merge area
@@ -637,8 +660,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        const bf16* __restrict__ v_cache, int cache_rows, const int* __restrict__ req_slot,
                        const int* __restrict__ block_table, int table_width, const int* __restrict__ dec_req,
                        const int* __restrict__ q_start, const int* __restrict__ ctx_len, float* __restrict__ partial,
-                       float* __restrict__ stats, int hq, int hkv, int page_size, float scale, int window, int keep_first,
-                       int split_size, int cluster, int n_parts, int row0, int* __restrict__ error) {
+                       float* __restrict__ stats, int hq, int hkv, int page_size, float scale, float softcap, int window,
+                       int keep_first, int split_size, int cluster, int n_parts, int row0, int* __restrict__ error) {
     CISR_TRACE_SCOPE(TRACE_ATTN_DECODE_TMA);
     extern __shared__ unsigned char smem_raw[];
     unsigned char* ring = reinterpret_cast<unsigned char*>(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);   // swizzle atoms are 1024-byte aligned
@@ -743,7 +766,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 #pragma unroll
     for (int kk = 0; kk < KD; ++kk)
         ldmatrix_x4(qf[kk], Qs + ((lane & 7) + 8 * ((lane >> 3) & 1)) * LDS + kk * 16 + 8 * (lane >> 4));
-    const float scale2 = scale * LOG2E;
+    const ScoreUnits units(scale, softcap);
 
     for (int t = warp, it = 0; t < n_tiles; t += 4, ++it) {
         const int slot = it % STAGES;
@@ -797,7 +820,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         for (int nt = 0; nt < TKT; ++nt) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                float v = s[nt][e] * scale2;
+                float v = units(s[nt][e]);
                 if (edge) {
                     const int kpos = k0 + nt * 8 + 2 * (lane & 3) + (e & 1);
                     if (kpos >= hi || kpos < lo || in_gap(run, kpos)) v = -INFINITY;
@@ -974,10 +997,10 @@ CISR_EXPORT int cisr_attn_prefill_tile() { return BM; }
 CISR_EXPORT int cisr_attn_prefill(const void* q, void* out, const void* k_cache, const void* v_cache,
                                   const int* req_slot, const int* block_table, int table_width, const int* tile_req,
                                   const int* tile_q0, int n_tiles, const int* q_start, const int* q_len,
-                                  const int* ctx_len, int hq, int hkv, int page_size, float scale, int window,
+                                  const int* ctx_len, int hq, int hkv, int page_size, float scale, float softcap, int window,
                                   int keep_first, float sink, const float* sink_heads, void* stream) {
     if (n_tiles <= 0) return 0;
-    if (hq % hkv) return -2;
+    if (hq % hkv || (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f)) return -2;
     const size_t smem = PREFILL_SMEM + sizeof(int) * ((size_t)table_width + 4);    // a tile's key range spans at most the table
     if (smem > 220 * 1024) return -3;
     static size_t configured = 0;
@@ -988,18 +1011,18 @@ CISR_EXPORT int cisr_attn_prefill(const void* q, void* out, const void* k_cache,
     }
     return launch_kernel(attn_prefill_mma_kernel, dim3(n_tiles, hq), dim3(PREFILL_THREADS), smem, (cudaStream_t)stream, g_pdl,
                          (const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache, req_slot, block_table,
-                         table_width, tile_req, tile_q0, q_start, q_len, ctx_len, hq, hkv, page_size, scale, window, keep_first, sink, sink_heads);
+                         table_width, tile_req, tile_q0, q_start, q_len, ctx_len, hq, hkv, page_size, scale, softcap, window, keep_first, sink, sink_heads);
 }
 
 CISR_EXPORT int cisr_attn_decode(const void* q, void* out, const void* k_cache, const void* v_cache,
                                  const int* req_slot, const int* block_table, int table_width, const int* dec_req,
                                  int n_dec, const int* q_start, const int* ctx_len, float* partial, float* stats, int hq,
-                                 int hkv, int page_size, float scale, int window, int keep_first, int split_size, int n_splits,
+                                 int hkv, int page_size, float scale, float softcap, int window, int keep_first, int split_size, int n_splits,
                                  int merge, float sink, const float* sink_heads, void* stream) {
     // merge == 0: the ranges' partial sums and statistics are left in `partial` and `stats` for the caller's own merge
     // (merge_proj.cu merges them in the prologue of the output projection); `out` is then not written.
     if (n_dec <= 0) return 0;
-    if (hq % hkv || split_size <= 0 || n_splits <= 0) return -2;
+    if (hq % hkv || split_size <= 0 || n_splits <= 0 || (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f)) return -2;
     const size_t smem = DEC_SMEM + sizeof(int) * ((size_t)split_size / page_size + 4);   // + the range's block table entries
     if (smem > 220 * 1024) return -3;
     static size_t configured = 0;
@@ -1014,7 +1037,7 @@ CISR_EXPORT int cisr_attn_decode(const void* q, void* out, const void* k_cache, 
         int status = launch_kernel(attn_decode_mma_kernel, dim3(n_dec, hkv, n_splits), dim3(DEC_THREADS), smem, s, g_pdl,
                                    (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, req_slot, block_table,
                                    table_width, dec_req, q_start, ctx_len, partial, stats, hq, hkv, page_size, scale,
-                                   window, keep_first, split_size, n_splits, row0);
+                                   softcap, window, keep_first, split_size, n_splits, row0);
         if (status) return status;
     }
     if (!merge) return 0;
@@ -1048,13 +1071,13 @@ CISR_EXPORT int cisr_attn_tma_init(int* error_flag) {
 CISR_EXPORT int cisr_attn_decode_tma(const void* q, void* out, const void* k_cache, const void* v_cache, int n_pages,
                                      const int* req_slot, const int* block_table, int table_width, const int* dec_req,
                                      int n_dec, const int* q_start, const int* ctx_len, float* partial, float* stats,
-                                     int hq, int hkv, int page_size, float scale, int window, int keep_first, int split_size,
+                                     int hq, int hkv, int page_size, float scale, float softcap, int window, int keep_first, int split_size,
                                      int n_splits, int merge, float sink, const float* sink_heads, void* stream) {
     // `sink` (-inf: none) is added to the denominator by the merge kernel, so the ranges are never merged inside a cluster then
     if (n_dec <= 0) return 0;
     if (!g_encode || !g_error) return -13;
     if (!merge && g_clusters) return -2;      // the caller's own merge needs every range's partial sum
-    if (hq % hkv || n_splits <= 0 || !cisr_attn_decode_tma_ok(page_size, split_size)) return -2;
+    if (hq % hkv || n_splits <= 0 || !cisr_attn_decode_tma_ok(page_size, split_size) || (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f)) return -2;
     const long long cache_rows = (long long)n_pages * hkv * page_size;
     if (cache_rows <= 0 || cache_rows >= (1ll << 31) || (((uintptr_t)k_cache | (uintptr_t)v_cache) & 15)) return -2;
     const int box_rows = page_size < TK ? page_size : TK;
@@ -1116,13 +1139,13 @@ CISR_EXPORT int cisr_attn_decode_tma(const void* q, void* out, const void* k_cac
             status = launch_kernel_cluster(attn_decode_tma_kernel<2>, dim3(n_dec, hkv, n_splits), dim3(DEC_THREADS), smem_deep, s, g_pdl, 1,
                                            map_k, map_v, (const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache,
                                            (int)cache_rows, req_slot, block_table, table_width,
-                                           dec_req, q_start, ctx_len, partial, stats, hq, hkv, page_size, scale, window, keep_first, split_size,
+                                           dec_req, q_start, ctx_len, partial, stats, hq, hkv, page_size, scale, softcap, window, keep_first, split_size,
                                            1, n_parts, row0, g_error);
         else
             status = launch_kernel_cluster(attn_decode_tma_kernel<1>, dim3(n_dec, hkv, n_splits), dim3(DEC_THREADS), smem, s, g_pdl, cluster,
                                            map_k, map_v, (const bf16*)q, (bf16*)out, (const bf16*)k_cache, (const bf16*)v_cache,
                                            (int)cache_rows, req_slot, block_table, table_width,
-                                           dec_req, q_start, ctx_len, partial, stats, hq, hkv, page_size, scale, window, keep_first, split_size,
+                                           dec_req, q_start, ctx_len, partial, stats, hq, hkv, page_size, scale, softcap, window, keep_first, split_size,
                                            cluster, n_parts, row0, g_error);
         if (status) return status;
     }

@@ -11,6 +11,7 @@
 //   k_cache[page][g][off] = [rotate(kn_g) | 0]
 //   v_cache[page][g][off] = [v_g | 0]  with v from its own columns, or (v_col < 0) the key as projected: with its bias,
 //                                      before norm and rotation; value_dim = key_dim then
+//   with `v_other` the value is blended first: v <- (1 - blend) v + blend v_other[t]   (v_other: rows `other_stride` apart)
 //
 // The first 2 * rot_half coordinates of a head turn; pairs are (i, i + rot_half) or, interleaved, (2i, 2i + 1).
 // The tables hold cos and sin per (token, pair), already multiplied by whatever factor the encoding wants.
@@ -57,7 +58,8 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
                       QT* __restrict__ q_out, CT* __restrict__ k_cache, CT* __restrict__ v_cache,
                       const int* __restrict__ token_req, const int* __restrict__ positions, const int* __restrict__ req_slot,
                       const int* __restrict__ block_table, int table_width, int page_size, int hq, int hkv, int key_dim,
-                      int value_dim, int D, int n_cols, int per_head, float temp_coef, double temp_every) {
+                      int value_dim, int D, int n_cols, int per_head, float temp_coef, double temp_every,
+                      const float* __restrict__ v_other, int other_stride, float blend) {
     extern __shared__ float row[];            // n_cols floats: the token's projection with its bias
     __shared__ float scratch[32];
     pdl_trigger();
@@ -67,6 +69,12 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
     pdl_wait();
     const float* src = proj + (size_t)t * row_stride;
     for (int i = threadIdx.x; i < n_cols; i += blockDim.x) row[i] = src[i] + (bias ? bias[i] : 0.f);
+    if (v_other) {       // a thread blends the columns it has just brought in
+        const float* other = v_other + (size_t)t * other_stride;
+        const int v_end = v_col + hkv * value_dim;
+        for (int i = threadIdx.x; i < v_end; i += blockDim.x)
+            if (i >= v_col) row[i] = (1.f - blend) * row[i] + blend * other[i - v_col];
+    }
     __syncthreads();
     const int nq = hq * key_dim, nk = hkv * key_dim;
     float inv_q = 1.f, inv_k = 1.f;
@@ -124,10 +132,11 @@ CISR_EXPORT int cisr_attention_rows(const float* proj, int row_stride, int k_col
                                     int interleaved, void* q_out, int q_dtype, void* k_cache, void* v_cache, int cache_dtype,
                                     const int* token_req, const int* positions, const int* req_slot, const int* block_table,
                                     int table_width, int page_size, int hq, int hkv, int key_dim, int value_dim, int D, int tokens,
-                                    int per_head, float temp_coef, double temp_every, void* stream) {
+                                    int per_head, float temp_coef, double temp_every, const float* v_other, int other_stride, float blend,
+                                    void* stream) {
     if (tokens <= 0) return 0;
     if (2 * rot_half > key_dim || rot_half < 0 || key_dim > D || value_dim > D || hq <= 0 || hkv <= 0) return -2;
-    if (v_col < 0 && value_dim != key_dim) return -2;
+    if (v_col < 0 && (value_dim != key_dim || v_other)) return -2;
     if (rot_half && (!cos_t || !sin_t)) return -2;
     if (temp_coef != 0.f && !(temp_every > 0.0)) return -2;
     const int n_cols = v_col >= 0 ? v_col + hkv * value_dim : k_col + hkv * key_dim;
@@ -148,7 +157,7 @@ CISR_EXPORT int cisr_attention_rows(const float* proj, int row_stride, int k_col
         return launch_kernel(attention_rows_kernel<QT, CT>, dim3(tokens), dim3(threads), smem, s, g_pdl, proj, row_stride, k_col, v_col, bias, \
                              q_norm, k_norm, eps, cos_t, sin_t, rot_half, interleaved, (QT*)q_out, (CT*)k_cache, (CT*)v_cache,   \
                              token_req, positions, req_slot, block_table, table_width, page_size, hq, hkv, key_dim, value_dim, D, n_cols,     \
-                             per_head, temp_coef, temp_every);                                                                                  \
+                             per_head, temp_coef, temp_every, v_other, other_stride, blend);                                                                                  \
     } while (0)
     if (q_dtype == CISR_BF16 && cache_dtype == CISR_BF16) CISR_ROWS(__nv_bfloat16, __nv_bfloat16);
     if (q_dtype == CISR_F32 && cache_dtype == CISR_F32) CISR_ROWS(float, float);

@@ -25,12 +25,16 @@
 // the sums and the maxima are float, P is rounded to bfloat16 once.  The keys a query sees, their split into the two
 // streams and their order do not depend on the batch: tiles start at multiples of 128 in absolute positions.
 //
+// With -DSOFTCAP=1 a score becomes cap tanh(score / cap) before the softmax (`softcap`; ignored otherwise): each thread
+// bends its scores as it takes them from tensor memory.
+//
 // Every wait on an mbarrier is bounded; a role whose wait ran out raises the CTA's abort flag and the device flag
 // (5), the other roles leave at their next wait, tensor memory is freed, and the host reports the failure.
 //
 // Parity: the online softmax of runtime/reference.py:18-27 and kernels/ops.cu:88-123 of the reference, tiled.
 // Cache layout: [pages, kv_heads, page_size, HEAD_DIM]; page sizes: multiples of 8 that divide 128 or are multiples of it.
 #include "tcgen05.cuh"
+#include "softcap.cuh"
 
 #ifndef HEAD_DIM
 #error "compile with -DHEAD_DIM=64 or 128"
@@ -78,7 +82,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ req_slot, const int* __restrict__ block_table, int table_width,
                             const int* __restrict__ tile_req, const int* __restrict__ tile_q0,
                             const int* __restrict__ q_start, const int* __restrict__ q_len,
-                            const int* __restrict__ ctx_len, int hq, int hkv, int page_size, float scale, int window,
+                            const int* __restrict__ ctx_len, int hq, int hkv, int page_size, float scale, float softcap, int window,
                             int keep_first, float sink_all, const float* __restrict__ sink_heads, int* __restrict__ error) {
     CISR_TRACE_SCOPE(TRACE_ATTN_PREFILL);
     extern __shared__ unsigned char smem_raw[];
@@ -246,7 +250,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int qpos = qpos0 + row;
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const uint32_t tmem_own = tmem_o + lane_base + (uint32_t)(group * D);     // this thread's row of its group's accumulator
-        const float scale2 = scale * LOG2E;
+        const float scale2 = SOFTCAP ? 1.f : scale * LOG2E;        // bent scores come in base-2 units
         auto softmax_sync = [&]() { asm volatile("bar.sync 1, %0;" ::"n"(SOFTMAX_THREADS) : "memory"); };
         float m_used = -INFINITY, l = 0.f;
         bool ok = true;
@@ -264,6 +268,11 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                 for (int c0 = 0; c0 < HALF; c0 += 32) tmem_load32_nowait(s_addr + c0, raw + c0);
                 tmem_load_wait();
+                if (SOFTCAP) {
+                    const Bend bend(scale, softcap);
+#pragma unroll
+                    for (int c = 0; c < HALF; ++c) raw[c] = __float_as_uint(bend(__uint_as_float(raw[c])));
+                }
                 if (edge) {
 #pragma unroll
                     for (int c = 0; c < HALF; ++c)
@@ -426,11 +435,11 @@ CISR_EXPORT int cisr_attn_tcgen05_ok(int page_size) {
 CISR_EXPORT int cisr_attn_prefill_tcgen05(const void* q, void* out, int n_tokens, const void* k_cache, const void* v_cache,
                                           int n_pages, const int* req_slot, const int* block_table, int table_width,
                                           const int* tile_req, const int* tile_q0, int n_tiles, const int* q_start,
-                                          const int* q_len, const int* ctx_len, int hq, int hkv, int page_size, float scale,
+                                          const int* q_len, const int* ctx_len, int hq, int hkv, int page_size, float scale, float softcap,
                                           int window, int keep_first, float sink, const float* sink_heads, void* stream) {
     if (n_tiles <= 0) return 0;
     if (!g_encode || !g_error) return -13;
-    if (hq % hkv || !cisr_attn_tcgen05_ok(page_size)) return -2;
+    if (hq % hkv || !cisr_attn_tcgen05_ok(page_size) || (SOFTCAP ? !(softcap > 0.f) : softcap != 0.f)) return -2;
     const long long cache_rows = (long long)n_pages * hkv * page_size;
     if (cache_rows <= 0 || cache_rows >= (1ll << 31) || (((uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)q | (uintptr_t)out) & 15)) return -2;
     const int box_rows = page_size < BN ? page_size : BN;
@@ -449,5 +458,5 @@ CISR_EXPORT int cisr_attn_prefill_tcgen05(const void* q, void* out, int n_tokens
     }
     return launch_kernel(attn_prefill_tcgen05_kernel, dim3(n_tiles, hq), dim3(THREADS), smem, (cudaStream_t)stream, g_pdl, map_q,
                          map_k, map_v, (bf16*)out, (int)cache_rows, req_slot, block_table, table_width, tile_req, tile_q0,
-                         q_start, q_len, ctx_len, hq, hkv, page_size, scale, window, keep_first, sink, sink_heads, g_error);
+                         q_start, q_len, ctx_len, hq, hkv, page_size, scale, softcap, window, keep_first, sink, sink_heads, g_error);
 }

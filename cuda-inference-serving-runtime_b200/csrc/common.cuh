@@ -64,6 +64,14 @@ __device__ __forceinline__ float gelu_tanh(float z) {
 // Activation of the gate in a gated feed-forward: silu (kind 0) or the tanh form of gelu (kind 1).
 __device__ __forceinline__ float gate_activation(float z, int kind) { return kind == 1 ? gelu_tanh(z) : z / (1.f + expf(-z)); }
 
+// The gated product of a feed-forward: act(g) u (kinds 0 and 1), or, kind 2, g' sigmoid(1.702 g') (u' + 1) with
+// g' = min(g, limit) and u' = u clamped to [-limit, limit].
+__device__ __forceinline__ float gated_product(float g, float u, int kind, float limit) {
+    if (kind != 2) return gate_activation(g, kind) * u;
+    g = fminf(g, limit);
+    return g / (1.f + expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+}
+
 // Sum over a whole block in a fixed order (warp shuffles, then warp 0 over the
 // per-warp sums), so a row's result does not depend on what else is in the batch.
 __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floats */) {

@@ -40,6 +40,62 @@ CISR_EXPORT int cisr_embedding(const void* table, int table_dtype, const int* id
     return launch_kernel(embedding_kernel<float>, dim3(tokens), dim3(128), 0, s, g_pdl, (const float*)table, ids, out, hidden, vocab, scale);
 }
 
+// The same with a second table, looked up by a hash of the token and the one before it in its sequence:
+//   out[t] = table[id] * scale + pairs[(before * mul_prev + id * mul_cur) mod buckets],
+// or, for a sequence's first token, the row behind the buckets.  The token before comes from the step itself, or, for
+// the first token that a request brings to the step, from `last` [slots]: the last token the request brought before.
+// That token's CTA, the only one that reads the slot's entry, then puts the request's newest token there.
+template <typename TT>
+__global__ void embedding_pairs_kernel(const TT* __restrict__ table, const TT* __restrict__ pairs, const int* __restrict__ ids,
+                                       const int* __restrict__ positions, const int* __restrict__ token_req,
+                                       const int* __restrict__ req_slot, const int* __restrict__ q_start, const int* __restrict__ q_len,
+                                       int* __restrict__ last, float* __restrict__ out, int hidden, int vocab, float scale, int buckets,
+                                       int mul_prev, int mul_cur) {
+    CISR_TRACE_SCOPE(TRACE_EMBEDDING);
+    __shared__ int bucket;
+    pdl_trigger();
+    pdl_wait();
+    CISR_TRACE_WAITED();
+    const int t = blockIdx.x;
+    const auto token = [&](int i) { const int v = ids[i]; return v < 0 ? 0 : (v >= vocab ? vocab - 1 : v); };
+    const int id = token(t);
+    if (threadIdx.x == 0) {
+        const int req = token_req[t], first = q_start[req];
+        int before;
+        if (t == first) {
+            int* kept = last + req_slot[req];
+            before = *kept;
+            *kept = token(first + q_len[req] - 1);
+        } else {
+            before = token(t - 1);
+        }
+        // the multipliers come reduced modulo the buckets, so the sum stays below 2^62
+        bucket = positions[t] == 0 ? buckets
+                                   : (int)(((long long)before * mul_prev + (long long)id * mul_cur) % buckets);
+    }
+    __syncthreads();
+    const TT* src = table + (size_t)id * hidden;
+    const TT* add = pairs + (size_t)bucket * hidden;
+    float* dst = out + (size_t)t * hidden;
+    for (int d = threadIdx.x; d < hidden; d += blockDim.x) dst[d] = to_float(src[d]) * scale + to_float(add[d]);
+}
+
+CISR_EXPORT int cisr_embedding_pairs(const void* table, const void* pairs, int table_dtype, const int* ids, const int* positions,
+                                     const int* token_req, const int* req_slot, const int* q_start, const int* q_len, int* last,
+                                     float* out, int tokens, int hidden, int vocab, float scale, int buckets, int mul_prev, int mul_cur,
+                                     void* stream) {
+    if (tokens <= 0) return 0;
+    if (buckets <= 0 || mul_prev < 0 || mul_prev >= buckets || mul_cur < 0 || mul_cur >= buckets) return -2;
+    cudaStream_t s = (cudaStream_t)stream;
+    const dim3 block(hidden >= 2048 ? 512 : 128);
+    if (table_dtype == CISR_BF16)
+        return launch_kernel(embedding_pairs_kernel<__nv_bfloat16>, dim3(tokens), block, 0, s, g_pdl, (const __nv_bfloat16*)table,
+                             (const __nv_bfloat16*)pairs, ids, positions, token_req, req_slot, q_start, q_len, last, out, hidden, vocab, scale,
+                             buckets, mul_prev, mul_cur);
+    return launch_kernel(embedding_pairs_kernel<float>, dim3(tokens), block, 0, s, g_pdl, (const float*)table, (const float*)pairs, ids,
+                         positions, token_req, req_slot, q_start, q_len, last, out, hidden, vocab, scale, buckets, mul_prev, mul_cur);
+}
+
 // ---------------------------------------------------------------- residual add + RMSNorm
 // For output row r: src = rows ? rows[r] : r;  v = x[src] + delta[src] * dscale;  (x[src] = v if write_back)
 // out[r] = v * rsqrt(mean(v^2) + eps) * w.  dscale (float, one per channel; null: 1) is a layer scale: the output of a
@@ -246,9 +302,10 @@ CISR_EXPORT int cisr_add_rmsnorm(float* x, const float* delta, const void* weigh
 }
 
 // ---------------------------------------------------------------- SwiGLU
-// gate_up [T, 2I] float: gate in columns [0, I), up in [I, 2I).  out = act(gate) * up, act silu (gate_act 0) or the tanh form of gelu (1).
+// gate_up [T, 2I] float: gate in columns [0, I), up in [I, 2I).  out = act(gate) * up, act silu (gate_act 0) or the tanh form of gelu (1), or the
+// clamped form (2; common.cuh: gated_product).
 template <typename OT>
-__global__ void swiglu_kernel(const float* __restrict__ gate_up, OT* __restrict__ out, int inter, int gate_act, size_t total) {
+__global__ void swiglu_kernel(const float* __restrict__ gate_up, OT* __restrict__ out, int inter, int gate_act, float gate_limit, size_t total) {
     CISR_TRACE_SCOPE(TRACE_SWIGLU);
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
@@ -256,16 +313,17 @@ __global__ void swiglu_kernel(const float* __restrict__ gate_up, OT* __restrict_
     const int c = (int)(i - t * inter);
     const float g = gate_up[t * 2 * inter + c];
     const float u = gate_up[t * 2 * inter + inter + c];
-    out[i] = from_float<OT>(gate_activation(g, gate_act) * u);
+    out[i] = from_float<OT>(gated_product(g, u, gate_act, gate_limit));
 }
 
-CISR_EXPORT int cisr_swiglu(const float* gate_up, void* out, int out_dtype, int tokens, int inter, int gate_act, void* stream) {
+CISR_EXPORT int cisr_swiglu(const float* gate_up, void* out, int out_dtype, int tokens, int inter, int gate_act, float gate_limit,
+                            void* stream) {
     const size_t total = (size_t)tokens * inter;
     if (!total) return 0;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == CISR_BF16) swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (__nv_bfloat16*)out, inter, gate_act, total);
-    else swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (float*)out, inter, gate_act, total);
+    if (out_dtype == CISR_BF16) swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (__nv_bfloat16*)out, inter, gate_act, gate_limit, total);
+    else swiglu_kernel<<<blocks, 256, 0, s>>>(gate_up, (float*)out, inter, gate_act, gate_limit, total);
     return launch_status();
 }
 

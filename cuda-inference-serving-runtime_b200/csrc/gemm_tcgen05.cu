@@ -449,13 +449,20 @@ CISR_EXPORT int cisr_gemm_tcgen05(const void* a, const void* w, float* out, int 
 }
 
 // w stacks gate rows [0, inter) over up rows [inter, 2 * inter); out (bfloat16 [m, inter]) = act(a gate^T) * (a up^T), act silu (gate_act 0)
-// or the tanh form of gelu (1).
-CISR_EXPORT int cisr_gemm_tcgen05_swiglu(const void* a, const void* w, void* out, int m, int inter, int k, int gate_act, void* stream) {
+// or the tanh form of gelu (1); gate_act 2: the clamped form, g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit).
+CISR_EXPORT int cisr_gemm_tcgen05_swiglu(const void* a, const void* w, void* out, int m, int inter, int k, int gate_act, float gate_limit,
+                                         void* stream) {
     if (m <= 0 || inter <= 0) return 0;
     if (!g_encode || !g_error) return -13;
     if (!operands_ok(a, w, k)) return -2;
     Epilogue ep = {};
     ep.out_bf16 = (bf16*)out; ep.inter = inter; ep.act = gate_act;
+    if (gate_act == 2) {
+        ep.limit = gate_limit; ep.alpha = 1.702f;
+        if (wide_tiles(m, (inter + 127) / 128))
+            return launch<256, 4, EPI_GATED>(a, w, ep, m, 2 * inter, k, (inter + 127) / 128, (cudaStream_t)stream);
+        return launch<128, 3, EPI_GATED>(a, w, ep, m, 2 * inter, k, (inter + 63) / 64, (cudaStream_t)stream);
+    }
     if (wide_tiles(m, (inter + 127) / 128)) {
         // 128 x 256 tiles, or 128 x 192 where their last round would be much emptier: 192 tiles of 256 columns on 148 SMs
         // are two rounds for 1.3 rounds of work, 256 tiles of 192 columns are two rounds of three quarters the length

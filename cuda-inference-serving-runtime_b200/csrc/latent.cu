@@ -129,11 +129,11 @@ CISR_EXPORT int cisr_latent_query(const float* q, int row_stride, int q_col, int
 }
 
 // ---------------------------------------------------------------- output gate
-// out[t, i] = values[t, i] * sigmoid(gate[t, gate_col + i]) (gate null: out = values), rounded to the storage type of
-// the output projection's operand.
+// out[t, i] = values[t, i] * sigmoid(gate[t, gate_col + i / per]) (gate null: out = values), rounded to the storage type of
+// the output projection's operand.  per 1: a gate per value; per = value_dim: one per head.
 template <typename CT>
 __global__ void latent_gate_kernel(const float* __restrict__ values, const float* __restrict__ gate, int gate_stride,
-                                   int gate_col, CT* __restrict__ out, int width, size_t total) {
+                                   int gate_col, int per, CT* __restrict__ out, int width, size_t total) {
     pdl_trigger();
     pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -141,22 +141,23 @@ __global__ void latent_gate_kernel(const float* __restrict__ values, const float
     float v = values[i];
     if (gate) {
         const size_t t = i / width;
-        const float g = gate[t * gate_stride + gate_col + (i - t * width)];
+        const float g = gate[t * gate_stride + gate_col + (int)(i - t * width) / per];
         v *= 1.f / (1.f + expf(-g));
     }
     out[i] = from_float<CT>(v);
 }
 
-CISR_EXPORT int cisr_latent_gate(const float* values, const float* gate, int gate_stride, int gate_col, void* out, int dtype,
+CISR_EXPORT int cisr_latent_gate(const float* values, const float* gate, int gate_stride, int gate_col, int per, void* out, int dtype,
                                  int tokens, int width, void* stream) {
     const size_t total = (size_t)tokens * width;
     if (!total) return 0;
+    if (per <= 0) return -2;
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid((unsigned)((total + 255) / 256));
     if (dtype == CISR_BF16)
-        return launch_kernel(latent_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, g_pdl, values, gate, gate_stride, gate_col,
+        return launch_kernel(latent_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, g_pdl, values, gate, gate_stride, gate_col, per,
                              (__nv_bfloat16*)out, width, total);
-    return launch_kernel(latent_gate_kernel<float>, grid, dim3(256), 0, s, g_pdl, values, gate, gate_stride, gate_col, (float*)out,
+    return launch_kernel(latent_gate_kernel<float>, grid, dim3(256), 0, s, g_pdl, values, gate, gate_stride, gate_col, per, (float*)out,
                          width, total);
 }
 
@@ -223,12 +224,12 @@ CISR_EXPORT int cisr_latent_absorb(const float* q, int row_stride, int q_col, in
 }
 
 // latent_values: the product with W_vup and the output gate in one launch.
-//   out[t, h * value_dim + j] = (sum_r mixed[t, h, r] * W_vup[h][j][r]) * sigmoid(gate[t, gate_col + h * value_dim + j])
+//   out[t, h * value_dim + j] = (sum_r mixed[t, h, r] * W_vup[h][j][r]) * sigmoid(gate[t, gate_col + (h * value_dim + j) / per])
 // mixed [tokens, heads, row_width] is the attention's weighted sum of cache rows (its first kv_rank columns count);
 // gate null: no gate.  A warp per output feature, its lanes striding over the latent.
 template <typename CT>
 __global__ void latent_values_kernel(const CT* __restrict__ mixed, int heads, int row_width, int kv_rank, const CT* __restrict__ v_up,
-                                     int value_dim, const float* __restrict__ gate, int gate_stride, int gate_col, CT* __restrict__ out) {
+                                     int value_dim, const float* __restrict__ gate, int gate_stride, int gate_col, int per, CT* __restrict__ out) {
     pdl_trigger();
     const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
     const int warp = blockIdx.z * n_warps + (threadIdx.x >> 5), all_warps = gridDim.z * n_warps;    // a warp has one feature when the grid is large enough
@@ -241,20 +242,21 @@ __global__ void latent_values_kernel(const CT* __restrict__ mixed, int heads, in
         acc = warp_sum(acc);
         if (lane == 0) {
             const int col = h * value_dim + j;
-            if (gate) acc *= 1.f / (1.f + expf(-gate[(size_t)t * gate_stride + gate_col + col]));
+            if (gate) acc *= 1.f / (1.f + expf(-gate[(size_t)t * gate_stride + gate_col + col / per]));
             out[(size_t)t * heads * value_dim + col] = from_float<CT>(acc);
         }
     }
 }
 
 CISR_EXPORT int cisr_latent_values(const void* mixed, int heads, int row_width, int kv_rank, const void* v_up, int value_dim,
-                                   const float* gate, int gate_stride, int gate_col, void* out, int dtype, int tokens, void* stream) {
+                                   const float* gate, int gate_stride, int gate_col, int per, void* out, int dtype, int tokens, void* stream) {
     if (tokens <= 0) return 0;
+    if (per <= 0) return -2;
     cudaStream_t s = (cudaStream_t)stream;
     const dim3 grid(tokens, heads, (value_dim + 7) / 8);
     if (dtype == CISR_BF16)
         return launch_kernel(latent_values_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, g_pdl, (const __nv_bfloat16*)mixed, heads, row_width,
-                             kv_rank, (const __nv_bfloat16*)v_up, value_dim, gate, gate_stride, gate_col, (__nv_bfloat16*)out);
+                             kv_rank, (const __nv_bfloat16*)v_up, value_dim, gate, gate_stride, gate_col, per, (__nv_bfloat16*)out);
     return launch_kernel(latent_values_kernel<float>, grid, dim3(256), 0, s, g_pdl, (const float*)mixed, heads, row_width, kv_rank,
-                         (const float*)v_up, value_dim, gate, gate_stride, gate_col, (float*)out);
+                         (const float*)v_up, value_dim, gate, gate_stride, gate_col, per, (float*)out);
 }

@@ -5,6 +5,7 @@
 //     v[d] = x[src][d] + norm_post(y[src])[d] * post_w[d] + (extra ? extra[src][d] : 0) + (vec ? vec[d] : 0)
 //     x_out[src][d] = v[d]                              (when `store`)
 //     h[r][d] = norm_pre(v)[d] * pre_w[d]               (h null: the stream only)
+//   (pre_kind 2: h[r][d] = v[d], for a layer that norms its sub-blocks' outputs only)
 //   norm(u) = (u - mean) / sqrt(var + eps) with var the mean squared deviation (kind 0), or u / sqrt(mean(u^2) + eps) (kind 1)
 //
 // y null: nothing is pending.  post_w is the output norm's weight, times the layer scale where a layer has one.  `extra` is
@@ -63,7 +64,7 @@ post_norm_kernel(const RowArgs a) {
             const int d = lane + width * i;
             if (live && d < runs) {
                 if (a.y) pw[EARLY ? i : 0] = load_run<VEC>(a.post_w + (size_t)d * VEC);
-                if (a.h) nw[EARLY ? i : 0] = load_run<VEC>(a.pre_w + (size_t)d * VEC);
+                if (a.h && a.pre_w) nw[EARLY ? i : 0] = load_run<VEC>(a.pre_w + (size_t)d * VEC);
             }
         }
     }
@@ -128,6 +129,15 @@ post_norm_kernel(const RowArgs a) {
         }
     }
     if (!a.h) return;
+    OT* out = reinterpret_cast<OT*>(a.h) + (size_t)r * hidden;
+    if (a.pre_kind == 2) {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int d = lane + width * i;
+            if (d < runs) store_run<VEC>(out + (size_t)d * VEC, v[i]);
+        }
+        return;
+    }
     const float mean = a.pre_kind == 0 ? total(sum) / (float)hidden : 0.f;
     float sq = 0.f;
 #pragma unroll
@@ -138,7 +148,6 @@ post_norm_kernel(const RowArgs a) {
         }
     }
     const float inv = 1.f / sqrtf(total(sq) / (float)hidden + a.pre_eps);
-    OT* out = reinterpret_cast<OT*>(a.h) + (size_t)r * hidden;
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         const int d = lane + width * i;
@@ -177,7 +186,7 @@ CISR_EXPORT int cisr_post_norm(const float* x, float* x_out, const float* y, con
                                const float* extra, const float* vec, const float* pre_w, float pre_eps, int pre_kind, void* h, int h_dtype,
                                const int* rows, int n_rows, int hidden, int store, void* stream) {
     if (n_rows <= 0) return 0;
-    if (hidden <= 0 || (y && !post_w) || (h && !pre_w) || post_kind < 0 || post_kind > 1 || pre_kind < 0 || pre_kind > 1) return -2;
+    if (hidden <= 0 || (y && !post_w) || (h && !pre_w && pre_kind != 2) || post_kind < 0 || post_kind > 1 || pre_kind < 0 || pre_kind > 2) return -2;
     RowArgs a;
     a.x = x; a.x_out = x_out; a.y = y; a.post_w = post_w; a.extra = extra; a.vec = vec; a.pre_w = pre_w; a.h = h; a.rows = rows;
     a.post_eps = post_eps; a.pre_eps = pre_eps; a.post_kind = post_kind; a.pre_kind = pre_kind; a.n_rows = n_rows; a.hidden = hidden; a.store = store;

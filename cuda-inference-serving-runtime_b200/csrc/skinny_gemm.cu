@@ -62,7 +62,8 @@ struct SkinnyArgs {
     int hq; int hkv; int dim;
     int accumulate;                                // PLAIN: out += product
     float out_mult;                                // PLAIN: the product is multiplied by it first (a constant factor of the residual branch)
-    int gate_act;                                  // SWIGLU: the gate's activation, 0 silu, 1 the tanh form of gelu
+    int gate_act;                                  // SWIGLU: the gate's activation, 0 silu, 1 the tanh form of gelu, 2 the clamped form
+    float gate_limit;                              // of the clamped form
 };
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -415,7 +416,7 @@ __global__ void __launch_bounds__(EPI == EPI_PLAIN ? 256 : 512) skinny_kernel(co
             }
             const float sc = inv_rms(mrow);
             g *= sc; u *= sc;
-            a.out_bf16[(size_t)mrow * a.inter + f] = __float2bfloat16_rn(gate_activation(g, a.gate_act) * u);
+            a.out_bf16[(size_t)mrow * a.inter + f] = __float2bfloat16_rn(gated_product(g, u, a.gate_act, a.gate_limit));
         }
     } else {
         const int dim = a.dim, hh = blockIdx.x;
@@ -540,7 +541,7 @@ CISR_EXPORT int cisr_skinny_gemm(const void* w, int n, int k, const void* act, c
                                  const float* sin_t, int rot_half, int interleaved, void* q_out, void* k_cache,
                                  void* v_cache, const int* positions, const int* token_req, const int* req_slot,
                                  const int* block_table, int table_width, int page_size, int hq, int hkv, int dim,
-                                 int accumulate, float out_mult, int gate_act, void* stream) {
+                                 int accumulate, float out_mult, int gate_act, float gate_limit, void* stream) {
     if (m <= 0) return 0;
     if (m > 64 || k % 8 || k <= 0 || n <= 0) return -2;
     if (epilogue == EPI_ROPE && (dim % 16 || dim > 256 || dim < 16 || n != (hq + 2 * hkv) * dim || 2 * rot_half > dim)) return -2;
@@ -548,7 +549,7 @@ CISR_EXPORT int cisr_skinny_gemm(const void* w, int n, int k, const void* act, c
     SkinnyArgs a;
     a.w = (const bf16*)w; a.n = n; a.k = k; a.act = (const bf16*)act; a.x = x; a.delta = delta; a.norm_w = norm_w;
     a.norm_w_bf16 = norm_w_dtype == CISR_BF16; a.eps = eps; a.x_out = x_out; a.rows = rows; a.m = m; a.rt = 1; a.ks = 1;
-    a.sums_in_smem = 0; a.accumulate = accumulate != 0 && epilogue == EPI_PLAIN; a.out_mult = out_mult; a.gate_act = gate_act;
+    a.sums_in_smem = 0; a.accumulate = accumulate != 0 && epilogue == EPI_PLAIN; a.out_mult = out_mult; a.gate_act = gate_act; a.gate_limit = gate_limit;
     a.out_f32 = out_f32; a.out_bf16 = (bf16*)out_bf16; a.inter = inter; a.cos_t = cos_t; a.sin_t = sin_t;
     a.rot_half = rot_half; a.interleaved = interleaved; a.q_out = (bf16*)q_out; a.k_cache = (bf16*)k_cache;
     a.v_cache = (bf16*)v_cache; a.positions = positions; a.token_req = token_req; a.req_slot = req_slot;

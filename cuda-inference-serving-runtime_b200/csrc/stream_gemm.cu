@@ -52,7 +52,8 @@ struct StreamArgs {
     int hq; int hkv; int dim;
     int accumulate;                                // PLAIN: out += product
     float out_mult;                                // PLAIN: the product is multiplied by it first (a constant factor of the residual branch)
-    int gate_act;                                  // SWIGLU: the gate's activation, 0 silu, 1 the tanh form of gelu
+    int gate_act;                                  // SWIGLU: the gate's activation, 0 silu, 1 the tanh form of gelu, 2 the clamped form
+    float gate_limit;                              // of the clamped form
     int grouped;                                   // the tensor map's last dimension counts 64-column groups: a stage is one box
     int stage_groups; int stage_bytes;             // k-slices (64 columns each) per stage, and the stage's size
 };
@@ -345,7 +346,7 @@ stream_kernel(const __grid_constant__ CUtensorMap map_w, const StreamArgs a, int
                 if (f >= a.inter) continue;
                 const int lr = (lf >> 3) * 16 + (lf & 7);
                 const float gate = summed(lr, mrow), up = summed(lr + 8, mrow);
-                a.out_bf16[(size_t)mrow * a.inter + f] = __float2bfloat16_rn(gate_activation(gate, a.gate_act) * up);
+                a.out_bf16[(size_t)mrow * a.inter + f] = __float2bfloat16_rn(gated_product(gate, up, a.gate_act, a.gate_limit));
             }
         } else if (usable) {
             const int per_head = a.dim / a.block_rows, hh = block / per_head, p = block - hh * per_head, half = a.block_rows / 2;
@@ -507,7 +508,7 @@ CISR_EXPORT int cisr_stream_gemm(const void* w, int n, int k, const void* act, c
                                  const float* sin_t, int rot_half, int interleaved, void* q_out, void* k_cache,
                                  void* v_cache, const int* positions, const int* token_req, const int* req_slot,
                                  const int* block_table, int table_width, int page_size, int hq, int hkv, int dim,
-                                 int accumulate, float out_mult, int gate_act, void* stream) {
+                                 int accumulate, float out_mult, int gate_act, float gate_limit, void* stream) {
     if (m <= 0) return 0;
     if (!g_encode || !g_error) return -13;
     if (m > 16 || k % 8 || k <= 0 || n <= 0 || ((uintptr_t)w & 15)) return -2;
@@ -519,7 +520,7 @@ CISR_EXPORT int cisr_stream_gemm(const void* w, int n, int k, const void* act, c
     StreamArgs a;
     a.n = n; a.k = k; a.act = (const bf16*)act; a.x = x; a.delta = delta; a.norm_w = norm_w;
     a.norm_w_bf16 = norm_w_dtype == CISR_BF16; a.eps = eps; a.x_out = x_out; a.rows = rows; a.m = m;
-    a.block_rows = 0; a.n_blocks = 0; a.stages = 0; a.accumulate = accumulate != 0 && epilogue == EPI_PLAIN; a.out_mult = out_mult; a.gate_act = gate_act;
+    a.block_rows = 0; a.n_blocks = 0; a.stages = 0; a.accumulate = accumulate != 0 && epilogue == EPI_PLAIN; a.out_mult = out_mult; a.gate_act = gate_act; a.gate_limit = gate_limit;
     a.out_f32 = out_f32; a.out_bf16 = (bf16*)out_bf16; a.inter = inter; a.cos_t = cos_t; a.sin_t = sin_t;
     a.rot_half = rot_half; a.interleaved = interleaved; a.q_out = (bf16*)q_out; a.k_cache = (bf16*)k_cache;
     a.v_cache = (bf16*)v_cache; a.positions = positions; a.token_req = token_req; a.req_slot = req_slot;

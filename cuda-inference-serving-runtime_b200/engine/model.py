@@ -132,8 +132,10 @@ class Model:
 
     def side_states(self) -> list:
         """Per run entry: the fixed-size state its mixer keeps besides its pages (None: none).  Always the entry's own,
-        also where the entry reads another entry's pages."""
-        return [getattr(self.layers[entry.layer].mixer, "side_state", lambda: None)() for entry in self.spec.run]
+        also where the entry reads another entry's pages.  Behind the last entry: the embedding's state, where it has one."""
+        states = [getattr(self.layers[entry.layer].mixer, "side_state", lambda: None)() for entry in self.spec.run]
+        own = self.embedding.side_state()
+        return states if own is None else states + [own]
 
     def make_cache(self, n_pages: int, page_size: int = 16, max_slots: int = 64) -> CacheManager:
         return CacheManager(self.cache_uses(), n_pages, page_size, max_slots, self.spec.max_positions,
@@ -158,7 +160,7 @@ class Model:
         """Run the step's tokens through every run entry; float logits [wanted rows, vocab]."""
         for part in self.step_beginners():
             part.begin_step(ctx)
-        stream = self.stream_class(self.embedding.forward(ctx.token_ids), self.spec.stream)
+        stream = self.stream_class(self.embedding.forward(ctx.token_ids, ctx, cache.side_state(len(self.spec.run))), self.spec.stream)
         for index, entry in enumerate(self.spec.run):
             if entry.add_embedding:
                 stream.add_embedding()

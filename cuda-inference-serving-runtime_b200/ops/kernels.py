@@ -74,6 +74,7 @@ def _elementwise():
     lib = load_library("elementwise.cu")
     if not getattr(lib, "_typed", False):
         lib.cisr_embedding.restype = ctypes.c_int
+        lib.cisr_embedding_pairs.restype = ctypes.c_int
         lib.cisr_add_rmsnorm.restype = ctypes.c_int
         lib.cisr_swiglu.restype = ctypes.c_int
         lib.cisr_rotary_tables.restype = ctypes.c_int
@@ -95,6 +96,24 @@ def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: 
         raise KernelError("embedding: shapes of ids, table and out disagree")
     _check(_elementwise().cisr_embedding(_p(table), dtype_code(table.dtype), _p(ids), _p(out), tokens, hidden,
                                          table.shape[0], ctypes.c_float(scale), _stream()), "embedding")
+    return out
+
+
+def embedding_pairs(table: torch.Tensor, pairs: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float, mul_prev: int, mul_cur: int,
+                    last: torch.Tensor, *, positions, token_req, req_slot, q_start, q_len) -> torch.Tensor:
+    """`embedding` plus a row of `pairs` [buckets + 1, hidden]: row (token before * mul_prev + token * mul_cur) mod buckets, or
+    the last row for a sequence's first token.  `last` int32 [slots, 1]: per request slot the newest token it has brought
+    so far; read for the first token a request brings to the step, and brought up to date."""
+    _need(table, None, "table", 2); _need(pairs, table.dtype, "pairs", 2); _need(out, torch.float32, "out", 2); _need(last, torch.int32, "last", 2)
+    for name, t in (("ids", ids), ("positions", positions), ("token_req", token_req), ("req_slot", req_slot), ("q_start", q_start), ("q_len", q_len)):
+        _need(t, torch.int32, name, 1)
+    tokens, hidden = out.shape
+    buckets = pairs.shape[0] - 1
+    if ids.numel() != tokens or positions.numel() != tokens or token_req.numel() != tokens or table.shape[1] != hidden or pairs.shape[1] != hidden or buckets < 1:
+        raise KernelError("embedding_pairs: shapes of ids, tables and out disagree")
+    _check(_elementwise().cisr_embedding_pairs(_p(table), _p(pairs), dtype_code(table.dtype), _p(ids), _p(positions), _p(token_req), _p(req_slot),
+                                               _p(q_start), _p(q_len), _p(last), _p(out), tokens, hidden, table.shape[0], ctypes.c_float(scale),
+                                               buckets, mul_prev % buckets, mul_cur % buckets, _stream()), "embedding_pairs")
     return out
 
 
@@ -155,16 +174,24 @@ def scale_(x: torch.Tensor, scale: float) -> torch.Tensor:
     return x
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}       # of the gate in a gated feed-forward
+# of the gate in a gated feed-forward; "gated_clamp" is g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gated_clamp": 2}
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, gate: str = "silu") -> torch.Tensor:
-    """out = act(gate_up[:, :I]) * gate_up[:, I:], act silu or the tanh form of gelu."""
+def _gate(gate: str, limit: Optional[float]) -> tuple:
+    """The gate's activation as the kernels take it: its number, and the limit of the clamped form."""
+    if (gate == "gated_clamp") != (limit is not None):
+        raise KernelError("a gate limit belongs to the gated_clamp activation, and to no other")
+    return GATE_ACTIVATIONS[gate], ctypes.c_float(limit or 0.0)
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, gate: str = "silu", limit: Optional[float] = None) -> torch.Tensor:
+    """out = act(gate_up[:, :I]) * gate_up[:, I:], act silu or the tanh form of gelu; or the clamped form (`GATE_ACTIVATIONS`)."""
     _need(gate_up, torch.float32, "gate_up", 2); _need(out, None, "out", 2)
     tokens, inter = out.shape
     if gate_up.shape != (tokens, 2 * inter):
         raise KernelError("swiglu: gate_up must be [tokens, 2 * intermediate]")
-    _check(_elementwise().cisr_swiglu(_p(gate_up), _p(out), dtype_code(out.dtype), tokens, inter, GATE_ACTIVATIONS[gate], _stream()), "swiglu")
+    _check(_elementwise().cisr_swiglu(_p(gate_up), _p(out), dtype_code(out.dtype), tokens, inter, *_gate(gate, limit), _stream()), "swiglu")
     return out
 
 
@@ -244,20 +271,32 @@ _attention_libs = {}
 TENSOR_CORE_MAX_HEAD_DIM = 128
 
 
-def _attention_source(head_dim: int, dtype: torch.dtype, kind: str):
-    """bfloat16 heads up to 128 wide run on the tensor cores; float, and wider heads, on the CUDA cores."""
+ATTENTION_MAX_HEAD_DIM = 512
+
+
+def _attention_source(head_dim: int, dtype: torch.dtype, kind: str, softcap: bool = False):
+    """bfloat16 heads up to 128 wide run on the tensor cores; float, and wider heads, on the CUDA cores.  `softcap`: the
+    build whose scores are bent (csrc/softcap.cuh)."""
     if kind not in ("auto", "simt"):
         raise KernelError(f"unknown attention kernel kind {kind!r}")
+    bent = {"SOFTCAP": 1} if softcap else {}
     if kind == "auto" and dtype == torch.bfloat16 and head_dim <= TENSOR_CORE_MAX_HEAD_DIM:
-        return "attention_mma.cu", {"HEAD_DIM": head_dim}
-    return "attention.cu", {"HEAD_DIM": head_dim, "STORAGE_BF16": dtype_code(dtype)}
+        return "attention_mma.cu", {"HEAD_DIM": head_dim, **bent}
+    return "attention.cu", {"HEAD_DIM": head_dim, "STORAGE_BF16": dtype_code(dtype), **bent}
 
 
-def attention_library(head_dim: int, dtype: torch.dtype, kind: str = "auto"):
-    if head_dim % 16 or not 16 <= head_dim <= 256:
-        raise KernelError(f"attention kernels take head sizes that are multiples of 16 from 16 to 256, not {head_dim}")
-    source, defines = _attention_source(head_dim, dtype, kind)
-    key = (source, head_dim, dtype)
+def _softcap(softcap) -> float:
+    """The cap as the kernels take it: 0 where scores stay as they are."""
+    if softcap is not None and not softcap > 0:
+        raise KernelError(f"softcap must be positive, not {softcap}")
+    return ctypes.c_float(softcap or 0.0)
+
+
+def attention_library(head_dim: int, dtype: torch.dtype, kind: str = "auto", softcap: bool = False):
+    if head_dim % 16 or not 16 <= head_dim <= ATTENTION_MAX_HEAD_DIM:
+        raise KernelError(f"attention kernels take head sizes that are multiples of 16 from 16 to {ATTENTION_MAX_HEAD_DIM}, not {head_dim}")
+    source, defines = _attention_source(head_dim, dtype, kind, softcap)
+    key = (source, head_dim, dtype, bool(softcap))
     lib = _attention_libs.get(key)
     if lib is None:
         lib = load_library(source, defines)
@@ -302,16 +341,16 @@ def _error_flag() -> torch.Tensor:
     return flag
 
 
-def attention_jobs(head_dim: int, dtype: torch.dtype):
+def attention_jobs(head_dim: int, dtype: torch.dtype, softcap: bool = False):
     """The build job of the attention library for this head size and storage type."""
-    source, defines = _attention_source(head_dim, dtype, "auto")
+    source, defines = _attention_source(head_dim, dtype, "auto", softcap)
     return (source, defines, ())
 
 
-def attention_tcgen05_jobs(head_dim: int, dtype: torch.dtype):
+def attention_tcgen05_jobs(head_dim: int, dtype: torch.dtype, softcap: bool = False):
     """The build jobs of the tcgen05 prompt attention, where this head size and storage type have one."""
     if dtype == torch.bfloat16 and head_dim in TCGEN05_HEAD_DIMS:
-        return [("attention_tcgen05.cu", {"HEAD_DIM": head_dim}, ())]
+        return [("attention_tcgen05.cu", {"HEAD_DIM": head_dim, **({"SOFTCAP": 1} if softcap else {})}, ())]
     return []
 
 
@@ -320,16 +359,16 @@ WIDE_TILE = 128                  # queries per tile of the tcgen05 prompt attent
 _attention_tcgen05_libs = {}
 
 
-def _attention_tcgen05(head_dim: int):
-    lib = _attention_tcgen05_libs.get(head_dim)
+def _attention_tcgen05(head_dim: int, softcap: bool = False):
+    lib = _attention_tcgen05_libs.get((head_dim, softcap))
     if lib is None:
-        lib = load_library("attention_tcgen05.cu", {"HEAD_DIM": head_dim})
+        lib = load_library("attention_tcgen05.cu", {"HEAD_DIM": head_dim, **({"SOFTCAP": 1} if softcap else {})})
         for name in ("cisr_attn_prefill_tcgen05", "cisr_attn_tcgen05_init", "cisr_attn_tcgen05_ok", "cisr_attn_tcgen05_tile"):
             getattr(lib, name).restype = ctypes.c_int
         assert lib.cisr_attn_tcgen05_tile() == WIDE_TILE
         _check(lib.cisr_attn_tcgen05_init(_p(_error_flag())), "tcgen05 attention init", own=0)
         lib.cisr_attn_tcgen05_set_pdl(int(_pdl_state["on"]))
-        _attention_tcgen05_libs[head_dim] = lib
+        _attention_tcgen05_libs[(head_dim, softcap)] = lib
     return lib
 
 
@@ -356,9 +395,9 @@ def _sink(sink, hq: Optional[int] = None) -> tuple:
 
 
 def attn_prefill_wide(q, out, k_cache, v_cache, req_slot, block_table, wide_req, wide_q0, q_start, q_len, ctx_len, hq, hkv,
-                      page_size, scale, window, sink=None, keep_first: int = 0) -> None:
+                      page_size, scale, window, sink=None, keep_first: int = 0, softcap: Optional[float] = None) -> None:
     """Attention of portions on tcgen05: q, out [tokens, hq, D]; tiles of 128 queries as (request, first query).
-    `sink`: see `_sink`.  `keep_first`: the sequence's first keys that stay in sight behind a window."""
+    `softcap`: a score s becomes softcap * tanh(s / softcap) before the softmax.  `sink`: see `_sink`.  `keep_first`: the sequence's first keys that stay in sight behind a window."""
     dim = k_cache.shape[-1]
     _need(q, torch.bfloat16, "q", 3); _need(out, torch.bfloat16, "out", 3); _need(k_cache, torch.bfloat16, "k_cache", 4)
     _need(v_cache, torch.bfloat16, "v_cache", 4)
@@ -367,38 +406,39 @@ def attn_prefill_wide(q, out, k_cache, v_cache, req_slot, block_table, wide_req,
         _need(t, torch.int32, name)
     if not attn_prefill_wide_ok(q, k_cache, page_size):
         raise KernelError("attn_prefill_wide: not a head size, page size or buffer for the tcgen05 attention")
-    lib = _attention_tcgen05(dim)
+    lib = _attention_tcgen05(dim, softcap is not None)
     _check(lib.cisr_attn_prefill_tcgen05(_p(q), _p(out), q.shape[0], _p(k_cache), _p(v_cache), k_cache.shape[0], _p(req_slot),
                                          _p(block_table), block_table.shape[1], _p(wide_req), _p(wide_q0), wide_req.numel(),
                                          _p(q_start), _p(q_len), _p(ctx_len), hq, hkv, page_size, ctypes.c_float(scale),
-                                         int(window or 0), int(keep_first or 0), *_sink(sink, hq), _stream()), "attn_prefill_wide")
+                                         _softcap(softcap), int(window or 0), int(keep_first or 0), *_sink(sink, hq), _stream()), "attn_prefill_wide")
 
 
 PREFILL_TILE = 64
 
 
 def attn_prefill(q, out, k_cache, v_cache, req_slot, block_table, tile_req, tile_q0, q_start, q_len, ctx_len, hq, hkv,
-                 page_size, scale, window, kind: str = "auto", sink=None, keep_first: int = 0) -> None:
+                 page_size, scale, window, kind: str = "auto", sink=None, keep_first: int = 0, softcap: Optional[float] = None) -> None:
     """Attention of portions: q, out [tokens, hq, D]; tiles list (request, first query of the tile).  Query i sees key
-    j <= i when window is None or i - j < window or j < keep_first."""
+    j <= i when window is None or i - j < window or j < keep_first.  `softcap`: a score s becomes
+    softcap * tanh(s / softcap) before the softmax."""
     dim = k_cache.shape[-1]
     _need(q, k_cache.dtype, "q"); _need(out, k_cache.dtype, "out"); _need(k_cache, None, "k_cache", 4)
     _need(v_cache, k_cache.dtype, "v_cache", 4)
     for name, t in (("req_slot", req_slot), ("block_table", block_table), ("tile_req", tile_req), ("tile_q0", tile_q0), ("q_start", q_start),
                     ("q_len", q_len), ("ctx_len", ctx_len)):
         _need(t, torch.int32, name)
-    lib = attention_library(dim, k_cache.dtype, kind)
+    lib = attention_library(dim, k_cache.dtype, kind, softcap is not None)
     _check(lib.cisr_attn_prefill(_p(q), _p(out), _p(k_cache), _p(v_cache), _p(req_slot), _p(block_table), block_table.shape[1],
                                  _p(tile_req), _p(tile_q0), tile_req.numel(), _p(q_start), _p(q_len), _p(ctx_len),
-                                 hq, hkv, page_size, ctypes.c_float(scale), int(window or 0), int(keep_first or 0), *_sink(sink, hq),
-                                 _stream()), "attn_prefill")
+                                 hq, hkv, page_size, ctypes.c_float(scale), _softcap(softcap), int(window or 0), int(keep_first or 0),
+                                 *_sink(sink, hq), _stream()), "attn_prefill")
 
 
 def attn_decode(q, out, k_cache, v_cache, req_slot, block_table, dec_req, n_dec, q_start, ctx_len, partial, stats, hq, hkv,
                 page_size, scale, window, split_size, n_splits, kind: str = "auto", staging: str = "auto", merge: bool = True,
-                sink=None, keep_first: int = 0) -> None:
+                sink=None, keep_first: int = 0, softcap: Optional[float] = None) -> None:
     """Attention of single new tokens, split over key ranges of `split_size`, merged into out.  `keep_first`: the
-    sequence's first keys that stay in sight behind a window.
+    sequence's first keys that stay in sight behind a window.  `softcap`: as for `attn_prefill`.
 
     `merge=False` (tensor-core kernels only) leaves the ranges' partial sums in `partial` and `stats` and does not write
     `out`: the caller merges them itself (`merge_out_proj`).
@@ -413,9 +453,10 @@ def attn_decode(q, out, k_cache, v_cache, req_slot, block_table, dec_req, n_dec,
         _need(t, torch.int32, name)
     if partial.numel() < n_dec * hq * n_splits * dim or stats.numel() < n_dec * hq * n_splits * 2:
         raise KernelError("attn_decode: scratch for partial sums is too small")
-    lib = attention_library(dim, k_cache.dtype, kind)
+    lib = attention_library(dim, k_cache.dtype, kind, softcap is not None)
     tail = [_p(req_slot), _p(block_table), block_table.shape[1], _p(dec_req), n_dec, _p(q_start), _p(ctx_len), _p(partial),
-            _p(stats), hq, hkv, page_size, ctypes.c_float(scale), int(window or 0), int(keep_first or 0), split_size, n_splits]
+            _p(stats), hq, hkv, page_size, ctypes.c_float(scale), _softcap(softcap), int(window or 0), int(keep_first or 0), split_size,
+            n_splits]
     if lib._tensor_core:
         tail.append(int(merge))
     elif not merge:
@@ -785,12 +826,14 @@ def attention_rows(proj: torch.Tensor, k_col: int, v_col: int, *, bias: Optional
                    k_norm: Optional[torch.Tensor], eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rot_half: int,
                    interleaved: bool, q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, token_req: torch.Tensor,
                    positions: torch.Tensor, req_slot: torch.Tensor, block_table: torch.Tensor, page_size: int, hq: int, hkv: int,
-                   key_dim: int, value_dim: int, norm_per_head: bool = False, q_temp=None) -> None:
+                   key_dim: int, value_dim: int, norm_per_head: bool = False, q_temp=None,
+                   other_values: Optional[torch.Tensor] = None, blend: float = 0.0) -> None:
     """proj float [tokens, cols] holds q at column 0, k at `k_col`, v at `v_col` (`v_col` < 0: the values are the keys as
     projected; columns behind those are another reader's).  Adds `bias` (float [cols]), norms q and k over their whole
     projection (`q_norm`, `k_norm`: float weights of that size, or None) or, with `norm_per_head`, each head by itself (weights
     of one head's size, shared by all), multiplies q by 1 + coef * ln(floor((position + 1) / every) + 1) where `q_temp` =
-    (coef, every) is given, rotates, pads the heads to the cache's width D, writes q_out [tokens, hq, D] and the key and value
+    (coef, every) is given, blends `other_values` (float rows [tokens, hkv * value_dim], may be columns of a wider tensor) into the
+    values where given, v <- (1 - blend) v + blend * other, rotates, pads the heads to the cache's width D, writes q_out [tokens, hq, D] and the key and value
     rows into their pages ([pages, hkv, page_size, D]).  See csrc/attention_rows.cu."""
     _need(proj, torch.float32, "proj", 2); _need(q_out, None, "q_out", 3); _need(k_cache, q_out.dtype, "k_cache", 4)
     _need(v_cache, q_out.dtype, "v_cache", 4)
@@ -810,12 +853,16 @@ def attention_rows(proj: torch.Tensor, k_col: int, v_col: int, *, bias: Optional
             raise KernelError("attention_rows: rotary tables must be [tokens, rot_half]")
     for name, t in (("token_req", token_req), ("positions", positions), ("req_slot", req_slot), ("block_table", block_table)):
         _need(t, torch.int32, name)
+    if other_values is not None and (other_values.dtype != torch.float32 or not other_values.is_cuda or v_col < 0
+                                     or other_values.shape != (tokens, hkv * value_dim) or other_values.stride(1) != 1):
+        raise KernelError("attention_rows: other_values must be float rows [tokens, hkv * value_dim], and need values of their own to join")
     _check(_attention_rows().cisr_attention_rows(
         _p(proj), cols, k_col, v_col, _p(bias), _p(q_norm), _p(k_norm), ctypes.c_float(eps), _p(cos if rot_half else None),
         _p(sin if rot_half else None), rot_half, int(interleaved), _p(q_out), dtype_code(q_out.dtype), _p(k_cache), _p(v_cache),
         dtype_code(k_cache.dtype), _p(token_req), _p(positions), _p(req_slot), _p(block_table), block_table.shape[1], page_size,
         hq, hkv, key_dim, value_dim, width, tokens, int(norm_per_head), ctypes.c_float(q_temp[0] if q_temp else 0.0),
-        ctypes.c_double(q_temp[1] if q_temp else 1.0), _stream()), "attention_rows")
+        ctypes.c_double(q_temp[1] if q_temp else 1.0), ctypes.c_void_p(other_values.data_ptr() if other_values is not None else 0),
+        other_values.stride(0) if other_values is not None else 0, ctypes.c_float(blend), _stream()), "attention_rows")
 
 
 def bias_add(out: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
@@ -1038,7 +1085,7 @@ def post_norm(x: torch.Tensor, *, y: Optional[torch.Tensor] = None, post_w: Opti
               x_out: Optional[torch.Tensor] = None, pre_w: Optional[torch.Tensor] = None, pre_eps: float = 0.0, pre_kind: str = "layer",
               h: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """v = x + norm(y) * post_w + extra + vector (y, extra, vector: each may be absent); x_out (may be x; None: not
-    stored) receives v, h = norm(v) * pre_w (None: not formed).  Norm kinds: "layer" (mean taken off) or "rms".  `rows` picks
+    stored) receives v, h = norm(v) * pre_w (None: not formed).  Norm kinds: "layer" (mean taken off) or "rms"; `pre_kind` "none": h = v as it is (no `pre_w`).  `rows` picks
     rows of x, y and extra that become rows of h (nothing is stored then).  See csrc/post_norm.cu."""
     _need(x, torch.float32, "x", 2)
     tokens, hidden = x.shape
@@ -1060,13 +1107,13 @@ def post_norm(x: torch.Tensor, *, y: Optional[torch.Tensor] = None, post_w: Opti
             raise KernelError("post_norm: rows are picked for reading only")
     if h is not None:
         _need(h, None, "h", 2)
-        if h.shape != (n_rows, hidden) or pre_w is None:
+        if h.shape != (n_rows, hidden) or (pre_w is None) != (pre_kind == "none"):
             raise KernelError("post_norm: h must have a row per row read, and needs pre_w")
     if y is not None and post_w is None:
         raise KernelError("post_norm: y needs post_w")
     lib = _loaded(_post_norm_state, "post_norm.cu", "post_norm", ("cisr_post_norm",))
     _check(lib.cisr_post_norm(_p(x), _p(x_out), _p(y), _p(post_w), ctypes.c_float(post_eps), NORM_KINDS[post_kind], _p(extra), _p(vector),
-                              _p(pre_w), ctypes.c_float(pre_eps), NORM_KINDS[pre_kind], _p(h), dtype_code(h.dtype) if h is not None else 0,
+                              _p(pre_w), ctypes.c_float(pre_eps), 2 if pre_kind == "none" else NORM_KINDS[pre_kind], _p(h), dtype_code(h.dtype) if h is not None else 0,
                               _p(rows), n_rows, hidden, int(x_out is not None), _stream()), "post_norm")
     return h
 
@@ -1393,17 +1440,18 @@ def latent_query(q: torch.Tensor, q_col: int, heads: int, plain_dim: int, cos: t
                                        _stream()), "latent_query")
 
 
-def latent_gate(values: torch.Tensor, gate: Optional[torch.Tensor], gate_col: int, out: torch.Tensor) -> torch.Tensor:
-    """out = values * sigmoid(gate[:, gate_col : gate_col + width]) (gate None: out = values), rounded to out's type."""
+def latent_gate(values: torch.Tensor, gate: Optional[torch.Tensor], gate_col: int, out: torch.Tensor, per: int = 1) -> torch.Tensor:
+    """out = values * sigmoid(gate[:, gate_col : gate_col + width]) (gate None: out = values), rounded to out's type.  `per`
+    neighbouring values share a gate (1: each has its own; the width of a head: one per head)."""
     _need(values, torch.float32, "values", 2); _need(out, None, "out", 2)
     tokens, width = values.shape
     if out.shape != values.shape:
         raise KernelError("latent_gate: out and values differ in shape")
     if gate is not None:
         _need(gate, torch.float32, "gate", 2)
-        if gate.shape[0] != tokens or gate_col + width > gate.shape[1]:
+        if gate.shape[0] != tokens or width % per or gate_col + width // per > gate.shape[1]:
             raise KernelError("latent_gate: the gate's columns lie outside its rows")
-    _check(_latent().cisr_latent_gate(_p(values), _p(gate), gate.shape[1] if gate is not None else 0, gate_col, _p(out),
+    _check(_latent().cisr_latent_gate(_p(values), _p(gate), gate.shape[1] if gate is not None else 0, gate_col, per, _p(out),
                                       dtype_code(out.dtype), tokens, width, _stream()), "latent_gate")
     return out
 
@@ -1427,9 +1475,11 @@ def latent_absorb(q: torch.Tensor, q_col: int, heads: int, plain_dim: int, cos: 
     return q_rows
 
 
-def latent_values(mixed: torch.Tensor, v_up: torch.Tensor, gate: Optional[torch.Tensor], gate_col: int, out: torch.Tensor) -> torch.Tensor:
+def latent_values(mixed: torch.Tensor, v_up: torch.Tensor, gate: Optional[torch.Tensor], gate_col: int, out: torch.Tensor,
+                  per: int = 1) -> torch.Tensor:
     """Few tokens: the per-head product with v_up ([heads, value_dim, kv_rank]) over the first kv_rank columns of
-    mixed [tokens, heads, row width], times sigmoid(gate[:, gate_col + ...]) when a gate is given, rounded to out's type."""
+    mixed [tokens, heads, row width], times sigmoid(gate[:, gate_col + ...]) when a gate is given
+    (`per` as for `latent_gate`), rounded to out's type."""
     _need(mixed, None, "mixed", 3); _need(v_up, mixed.dtype, "v_up", 3); _need(out, mixed.dtype, "out", 2)
     tokens, heads, row_width = mixed.shape
     _, value_dim, kv_rank = v_up.shape
@@ -1437,10 +1487,10 @@ def latent_values(mixed: torch.Tensor, v_up: torch.Tensor, gate: Optional[torch.
         raise KernelError("latent_values: shapes disagree")
     if gate is not None:
         _need(gate, torch.float32, "gate", 2)
-        if gate.shape[0] != tokens or gate_col + heads * value_dim > gate.shape[1]:
+        if gate.shape[0] != tokens or (heads * value_dim) % per or gate_col + heads * value_dim // per > gate.shape[1]:
             raise KernelError("latent_values: the gate's columns lie outside its rows")
     _check(_latent().cisr_latent_values(_p(mixed), heads, row_width, kv_rank, _p(v_up), value_dim, _p(gate),
-                                        gate.shape[1] if gate is not None else 0, gate_col, _p(out), dtype_code(out.dtype), tokens,
+                                        gate.shape[1] if gate is not None else 0, gate_col, per, _p(out), dtype_code(out.dtype), tokens,
                                         _stream()), "latent_values")
     return out
 
@@ -1781,7 +1831,7 @@ def set_pdl(on: bool) -> None:
         _ffn_rows_state["lib"].cisr_ffn_rows_set_pdl(int(on))
     if "lib" in _tcgen05_state:
         _tcgen05_state["lib"].cisr_gemm_tcgen05_set_pdl(int(on))
-    for (source, _, _), lib in list(_attention_libs.items()):
+    for (source, *_), lib in list(_attention_libs.items()):
         if source == "attention_mma.cu":
             lib.cisr_attn_set_pdl(int(on))
     _pdl_state["on"] = bool(on)
@@ -1816,7 +1866,7 @@ def skinny_gemm(w: torch.Tensor, tokens: int, *, act: Optional[torch.Tensor] = N
                 delta: Optional[torch.Tensor] = None, norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
                 x_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, epilogue: int = EPI_PLAIN,
                 out: Optional[torch.Tensor] = None, rope: Optional[dict] = None, kind: str = "auto",
-                accumulate: bool = False, out_mult: float = 1.0, gate: str = "silu") -> None:
+                accumulate: bool = False, out_mult: float = 1.0, gate: str = "silu", gate_limit: Optional[float] = None) -> None:
     """out = prologue(input) @ w^T with a fused epilogue; see csrc/skinny_gemm.cu and csrc/stream_gemm.cu.
 
     `kind`: "latency" (skinny_gemm.cu: a CTA per 16 output rows, weights straight to registers), "stream"
@@ -1827,7 +1877,7 @@ def skinny_gemm(w: torch.Tensor, tokens: int, *, act: Optional[torch.Tensor] = N
     optional `x_out` receiving x + delta, optional `rows` picking rows of x).  PLAIN writes float `out`
     [tokens, N], or with `accumulate` adds the product to what `out` holds (the residual stream), in both cases times
     `out_mult` (a constant factor of the residual branch); SWIGLU writes bfloat16 `out` [tokens, N / 2] with the activation
-    `gate` ("silu" or "gelu_tanh") on the gate; ROPE takes the `rope` dict (cos, sin, rot_half,
+    `gate` ("silu", "gelu_tanh", or "gated_clamp" with its `gate_limit`) on the gate; ROPE takes the `rope` dict (cos, sin, rot_half,
     interleaved, q_out, k_cache, v_cache, positions, token_req, req_slot, block_table, page_size, hq, hkv, dim).
     """
     _need(w, torch.bfloat16, "w", 2)
@@ -1872,7 +1922,7 @@ def skinny_gemm(w: torch.Tensor, tokens: int, *, act: Optional[torch.Tensor] = N
             int(bool(r.get("interleaved", False))), _p(r.get("q_out")), _p(r.get("k_cache")), _p(r.get("v_cache")),
             _p(r.get("positions")), _p(r.get("token_req")), _p(r.get("req_slot")), _p(r.get("block_table")),
             r["block_table"].shape[1] if rope else 0, int(r.get("page_size", 0)), int(r.get("hq", 0)), int(r.get("hkv", 0)),
-            int(r.get("dim", 0)), int(bool(accumulate)), ctypes.c_float(out_mult), GATE_ACTIVATIONS[gate], _stream())
+            int(r.get("dim", 0)), int(bool(accumulate)), ctypes.c_float(out_mult), *_gate(gate, gate_limit), _stream())
     if (accumulate or out_mult != 1.0) and epilogue != EPI_PLAIN:
         raise KernelError("skinny_gemm: only the plain epilogue adds into its output or multiplies it")
     if kind not in ("auto", "latency", "stream"):
@@ -1953,15 +2003,15 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate
     return out
 
 
-def gemm_tcgen05_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: str = "silu") -> torch.Tensor:
-    """out (bfloat16 [M, I]) = act(a @ w[:I]^T) * (a @ w[I:]^T): the product with the gated activation (silu, or the tanh
-    form of gelu) as its epilogue."""
+def gemm_tcgen05_swiglu(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: str = "silu", limit: Optional[float] = None) -> torch.Tensor:
+    """out (bfloat16 [M, I]) = act(a @ w[:I]^T) * (a @ w[I:]^T): the product with the gated activation (silu, the tanh
+    form of gelu, or the clamped form) as its epilogue."""
     _need(a, torch.bfloat16, "a", 2); _need(w, torch.bfloat16, "w", 2); _need(out, torch.bfloat16, "out", 2)
     m, k = a.shape
     inter = out.shape[1]
     if w.shape != (2 * inter, k) or out.shape[0] != m:
         raise KernelError(f"gemm swiglu: shapes a{tuple(a.shape)} w{tuple(w.shape)} out{tuple(out.shape)} disagree")
-    _check(_tcgen05().cisr_gemm_tcgen05_swiglu(_p(a), _p(w), _p(out), m, inter, k, GATE_ACTIVATIONS[gate], _stream()), "gemm_tcgen05_swiglu")
+    _check(_tcgen05().cisr_gemm_tcgen05_swiglu(_p(a), _p(w), _p(out), m, inter, k, *_gate(gate, limit), _stream()), "gemm_tcgen05_swiglu")
     return out
 
 
@@ -2087,6 +2137,7 @@ def _describe_gemm(a, w, *rest, **kw):
 
 _DESCRIBE = {
     "embedding": lambda table, ids, out, scale=1.0: (int(out.shape[0]), int(out.shape[1])),
+    "embedding_pairs": lambda table, pairs, ids, out, *a, **kw: (int(out.shape[0]), int(out.shape[1])),
     "add_rmsnorm": lambda x, delta, weight, eps, out, rows=None, write_back=True, delta_scale=None: (int(out.shape[0]), int(out.shape[1]), delta is not None),
     "stream_add": lambda x, *a, **kw: (int(x.shape[0]), int(x.shape[1])),
     "scale_": lambda x, scale: (int(x.numel()),),
@@ -2106,7 +2157,7 @@ _DESCRIBE = {
     "gemm_tcgen05_grouped_gated": lambda a, w, out, tile_group, limit, rows_in_use=None:
         (int(rows_in_use or a.shape[0]), int(w.shape[0]), int(w.shape[1]), int(w.shape[2])),
     "gemm_heads": lambda a, w, out, w_is_nk: (int(a.shape[0]), int(w.shape[0]), int(w.shape[1]), int(w.shape[2])),
-    "swiglu": lambda gate_up, out, gate="silu": (int(out.shape[0]), int(out.shape[1])),
+    "swiglu": lambda gate_up, out, gate="silu", limit=None: (int(out.shape[0]), int(out.shape[1])),
     "rotary_tables": lambda positions, inv_freq, cos, sin, magnitude=1.0: (int(cos.shape[0]), int(cos.shape[1])),
     "hyper_mix_norm": lambda source, streams, n_streams, **kw:
         (int(streams.shape[0] if kw.get("h") is None else kw["h"].shape[0]), int(n_streams), int(streams.shape[2]), kw.get("y") is not None,

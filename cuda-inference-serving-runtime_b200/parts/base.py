@@ -181,8 +181,13 @@ class FeedForward(Part):
 
 
 class Embedding(Part):
-    def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
-        """int32 [tokens] -> float residual stream [tokens, hidden]."""
+    def side_state(self) -> Optional[CacheUse]:
+        """The fixed-size state per request that the embedding keeps (None: none): what it must remember of the tokens
+        that earlier steps brought."""
+        return None
+
+    def forward(self, token_ids: torch.Tensor, ctx=None, state: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """int32 [tokens] -> float residual stream [tokens, hidden]; `state` [slots, ...] where `side_state` asks for one."""
         raise NotImplementedError
 
 

@@ -1,4 +1,4 @@
-"""Token embedding and the output head.
+"""Token embedding (with, where a model has one, a second table looked up by pairs of tokens) and the output head.
 
 Parity: runtime/model.py:105 (lookup, no scaling) and runtime/model.py:120 (logits =
 norm(x) @ head^T, no bias, no scaling); a tied head is the embedding table itself
@@ -10,6 +10,7 @@ from typing import Dict
 
 import torch
 
+from ..config.spec import CacheUse
 from ..ops import kernels
 from .base import EMBEDDINGS, HEADS, Embedding, Head, Part, TensorNeed, register
 from .linear import linear
@@ -17,7 +18,10 @@ from .linear import linear
 
 @register(EMBEDDINGS, "token_embedding")
 class TokenEmbedding(Embedding):
-    """params: vocab_size, hidden_size; scale (the looked-up row is multiplied by it, default 1); weight_name."""
+    """params: vocab_size, hidden_size; scale (the looked-up row is multiplied by it, default 1); weight_name; pairs (None, or
+    {"buckets", "mul_prev", "mul_cur", "weight_name"}: a second table of buckets + 1 rows is added, row (token before *
+    mul_prev + token * mul_cur) mod buckets, and the last row for a sequence's first token.  The newest token of each
+    request is then part of its state)."""
 
     def __init__(self, spec, dtype):
         super().__init__(spec, dtype)
@@ -25,20 +29,33 @@ class TokenEmbedding(Embedding):
         self.hidden = int(spec["hidden_size"])
         self.scale = float(spec.get("scale", 1.0))
         self.weight_name = spec.get("weight_name", "weight")
-        self.table = None
+        self.pairs = dict(spec.get("pairs") or {})
+        self.table = self.pair_table = None
 
     def tensor_needs(self) -> Dict[str, TensorNeed]:
-        return {self.weight_name: TensorNeed((self.vocab, self.hidden))}
+        needs = {self.weight_name: TensorNeed((self.vocab, self.hidden))}
+        if self.pairs:
+            needs[self.pairs["weight_name"]] = TensorNeed((int(self.pairs["buckets"]) + 1, self.hidden))
+        return needs
 
     def load(self, tensors):
         self.table = tensors[self.weight_name]
+        if self.pairs:
+            self.pair_table = tensors[self.pairs["weight_name"]]
 
     def kernel_jobs(self):
         return [("elementwise.cu", {}, ())]
 
-    def forward(self, token_ids):
+    def side_state(self):
+        return CacheUse("state", state_shape=(1,), state_dtype="int32") if self.pairs else None
+
+    def forward(self, token_ids, ctx=None, state=None):
         out = torch.empty((token_ids.numel(), self.hidden), dtype=torch.float32, device=token_ids.device)
-        return kernels.embedding(self.table, token_ids, out, self.scale)
+        if not self.pairs:
+            return kernels.embedding(self.table, token_ids, out, self.scale)
+        return kernels.embedding_pairs(self.table, self.pair_table, token_ids, out, self.scale, int(self.pairs["mul_prev"]), int(self.pairs["mul_cur"]),
+                                       state, positions=ctx.positions, token_req=ctx.token_req, req_slot=ctx.req_slot, q_start=ctx.q_start,
+                                       q_len=ctx.q_len)
 
 
 @register(HEADS, "linear_head")

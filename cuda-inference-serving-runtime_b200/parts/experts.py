@@ -11,7 +11,8 @@
               or gated ("gated_clamp"):
               g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), W_down (g sigmoid(1.702 g) (u + 1))
     identity  the last `identity` router outputs have no matrices: such an expert's output is h itself
-    shared    an expert of the same form (its own width and limit) that every token uses, times sigmoid(w_sg . h)
+    shared    an expert of the same form (its own width and limit) that every token uses, times sigmoid(w_sg . h) where it
+              has a `w_sg`
     output    the weighted sum of the chosen experts' outputs (+ the shared expert's)
 
 The experts' matrices are stacked at load ([experts, ff, hidden] and [experts, hidden, ff]) so one launch serves
@@ -25,6 +26,7 @@ import torch
 
 from ..ops import kernels
 from .base import FEED_FORWARDS, FeedForward, TensorNeed, register
+from .feedforward import gated_product, pad_columns
 from .linear import linear, linear_add
 
 ACTIVATIONS = ("relu_squared", "gelu", "gated_clamp")
@@ -38,7 +40,7 @@ class RoutedExperts(FeedForward):
     """params: hidden_size, expert_size, experts, top, groups, keep, route_scale, activation, names (local tensor names:
     router, and up / down (/ gate) with {} for the expert's number); scores ("sigmoid" or "softmax"), choice_bias (bool),
     identity (router outputs beyond `experts` without matrices), limit (of the gated activation), shared (None, or
-    {"size", "limit"}: the shared expert), renormalize (bool: the chosen scores are divided by their sum)."""
+    {"size", "limit", "scaled" (default True: it has a w_sg)}: the shared expert), renormalize (bool: the chosen scores are divided by their sum)."""
 
     applies_output_scale = True      # forward(h, ctx, out_scale): a per-channel layer scale is the epilogue of the last kernel
 
@@ -62,6 +64,7 @@ class RoutedExperts(FeedForward):
         shared = spec.get("shared")
         self.shared_size = int(shared["size"]) if shared else 0
         self.shared_limit = float(shared["limit"]) if shared else None
+        self.shared_scaled = bool(shared.get("scaled", True)) if shared else False
         if self.scores not in ("sigmoid", "softmax"):
             raise ValueError(f"router scores {self.scores!r} are not implemented; known: sigmoid, softmax")
         if self.identity and self.groups:
@@ -91,7 +94,8 @@ class RoutedExperts(FeedForward):
             needs[self.names["shared_gate"]] = TensorNeed((self.shared_size, self.hidden))
             needs[self.names["shared_up"]] = TensorNeed((self.shared_size, self.hidden))
             needs[self.names["shared_down"]] = TensorNeed((self.hidden, self.shared_size))
-            needs[self.names["shared_scale"]] = TensorNeed((1, self.hidden))
+            if self.shared_scaled:
+                needs[self.names["shared_scale"]] = TensorNeed((1, self.hidden))
         return needs
 
     def load(self, tensors):
@@ -106,9 +110,9 @@ class RoutedExperts(FeedForward):
             self.up = torch.stack([tensors[n["up"].format(e)] for e in range(self.experts)]).contiguous()
         self.down = torch.stack([tensors[n["down"].format(e)] for e in range(self.experts)]).contiguous()
         if self.shared_size:
-            # gate rows, up rows, then the row whose product with h is the logit of the shared expert's per-token factor
-            self.shared_in = torch.cat((tensors[n["shared_gate"]], tensors[n["shared_up"]], tensors[n["shared_scale"]]), dim=0).contiguous()
-            from .feedforward import pad_columns
+            # gate rows, up rows, then (scaled) the row whose product with h is the logit of the shared expert's per-token factor
+            rows = ("shared_gate", "shared_up") + (("shared_scale",) if self.shared_scaled else ())
+            self.shared_in = torch.cat([tensors[n[row]] for row in rows], dim=0).contiguous()
             self.shared_down = pad_columns(tensors[n["shared_down"]], 8)
 
     def kernel_jobs(self):
@@ -128,10 +132,13 @@ class RoutedExperts(FeedForward):
 
     def shared_expert(self, h: torch.Tensor, into: torch.Tensor) -> torch.Tensor:
         """into += sigmoid(w_sg . h) * W_down act(W_gate h, W_up h): the factor is applied to the activations (the product
-        after it is linear), in float, before their one rounding; the add is the last product's epilogue."""
+        after it is linear), in float, before their one rounding; the add is the last product's epilogue.  Without a factor
+        the activation is the first product's epilogue where the kernels have it."""
+        if not self.shared_scaled and self.shared_down.shape[1] == self.shared_size:
+            return linear_add(gated_product(h, self.shared_in, "gated_clamp", self.shared_limit), self.shared_down, into)
         sums = linear(h, self.shared_in)                   # float [tokens, gate | up | factor logit]
         act = torch.empty((h.shape[0], self.shared_down.shape[1]), dtype=self.dtype, device=h.device)
-        kernels.gated_clamp(sums, self.shared_size, self.shared_limit, act, scale_col=2 * self.shared_size)
+        kernels.gated_clamp(sums, self.shared_size, self.shared_limit, act, scale_col=2 * self.shared_size if self.shared_scaled else -1)
         return linear_add(act, self.shared_down, into)
 
     def forward(self, h, ctx, out_scale=None):

@@ -1,4 +1,5 @@
-"""SwiGLU feed-forward: down(silu(gate(h)) * up(h)), or with the tanh form of gelu on the gate.
+"""SwiGLU feed-forward: down(silu(gate(h)) * up(h)), or with the tanh form of gelu on the gate, or with the clamped form
+g' sigmoid(1.702 g') (u' + 1) of gate and up, g' = min(g, limit), u' = clamp(u, -limit, limit).
 
 Parity: runtime/model.py:116-119, kernels/execution.cu:7-10.  gate_proj and up_proj
 are stacked into one [2I, H] matrix at load so one product serves both.
@@ -16,8 +17,8 @@ from .linear import as_tensor, linear, linear_to_stream, norm_fusable
 
 @register(FEED_FORWARDS, "swiglu")
 class SwiGLU(FeedForward):
-    """params: hidden_size, intermediate_size; activation of the gate ("silu", the default, or "gelu_tanh"); names (local
-    tensor names of gate, up, down)."""
+    """params: hidden_size, intermediate_size; activation of the gate ("silu", the default, "gelu_tanh", or "gated_clamp" with
+    its `limit`); names (local tensor names of gate, up, down)."""
 
     accepts_pending_norm = True
 
@@ -29,6 +30,7 @@ class SwiGLU(FeedForward):
         self.activation = spec.get("activation", "silu")
         if self.activation not in kernels.GATE_ACTIVATIONS:
             raise ValueError(f"unknown gate activation {self.activation!r}")
+        self.limit = float(spec["limit"]) if self.activation == "gated_clamp" else None
         self.gate_up = None
         self.down = None
 
@@ -46,26 +48,30 @@ class SwiGLU(FeedForward):
                 + (kernels.skinny_jobs() if self.dtype == torch.bfloat16 else []))
 
     def forward(self, h, ctx):
-        h0 = h
-        tokens = h.x.shape[0] if not isinstance(h, torch.Tensor) else h.shape[0]
-        device = h.x.device if not isinstance(h, torch.Tensor) else h.device
-        act = torch.empty((tokens, self.inter), dtype=self.dtype, device=device)
-        if kernels.skinny_ok(tokens, self.gate_up):
-            # few tokens: (norm,) gate and up products and the activation in one launch
-            if norm_fusable(h, tokens, self.gate_up):
-                x_out = h.new_stream_buffer()
-                kernels.skinny_gemm(self.gate_up, tokens, x=h.x, delta=h.delta, norm_w=h.weight, eps=h.eps, x_out=x_out,
-                                    epilogue=kernels.EPI_SWIGLU, out=act, gate=self.activation)
-                h.done(x_out)
-            else:
-                kernels.skinny_gemm(self.gate_up, tokens, act=as_tensor(h), epilogue=kernels.EPI_SWIGLU, out=act, gate=self.activation)
+        return linear_to_stream(gated_product(h, self.gate_up, self.activation, self.limit), self.down, h)
+
+
+def gated_product(h, gate_up: torch.Tensor, activation: str, limit=None) -> torch.Tensor:
+    """act(h W_gate^T, h W_up^T) for the stacked matrices gate_up [2I, H], [tokens, I] in their type; `h` a tensor or a
+    pending norm."""
+    tokens = h.x.shape[0] if not isinstance(h, torch.Tensor) else h.shape[0]
+    act = torch.empty((tokens, gate_up.shape[0] // 2), dtype=gate_up.dtype, device=gate_up.device)
+    if kernels.skinny_ok(tokens, gate_up):
+        # few tokens: (norm,) gate and up products and the activation in one launch
+        gate = dict(epilogue=kernels.EPI_SWIGLU, out=act, gate=activation, gate_limit=limit)
+        if norm_fusable(h, tokens, gate_up):
+            x_out = h.new_stream_buffer()
+            kernels.skinny_gemm(gate_up, tokens, x=h.x, delta=h.delta, norm_w=h.weight, eps=h.eps, x_out=x_out, **gate)
+            h.done(x_out)
         else:
-            hn = as_tensor(h)
-            if kernels.tcgen05_ok(hn, self.gate_up):
-                kernels.gemm_tcgen05_swiglu(hn, self.gate_up, act, gate=self.activation)      # many tokens: SwiGLU is the product's epilogue
-            else:
-                kernels.swiglu(linear(hn, self.gate_up), act, gate=self.activation)
-        return linear_to_stream(act, self.down, h0)
+            kernels.skinny_gemm(gate_up, tokens, act=as_tensor(h), **gate)
+    else:
+        hn = as_tensor(h)
+        if kernels.tcgen05_ok(hn, gate_up):
+            kernels.gemm_tcgen05_swiglu(hn, gate_up, act, gate=activation, limit=limit)      # many tokens: the activation is the product's epilogue
+        else:
+            kernels.swiglu(linear(hn, gate_up), act, gate=activation, limit=limit)
+    return act
 
 
 def pad_columns(w: torch.Tensor, multiple: int) -> torch.Tensor:

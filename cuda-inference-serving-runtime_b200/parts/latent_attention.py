@@ -9,7 +9,7 @@ Per token, with input h (the normed stream):
     per head     key_h = [W_kup_h c | k_rot],  value_h = W_vup_h c
     scores       (q_h . key_h) * scale over the keys j <= i (with `window`: i - j < window), softmax (with `sink`: one more
                  term exp(sink_h) per head in the denominator, with no key and no value), out_h = sum of weights * value_h
-    output       W_out (concatenated heads [* sigmoid(W_gate h)])
+    output       W_out (concatenated heads [* sigmoid(W_gate h)])           W_gate: a row per value, or (gate "head") per head
 
 `shared_kv`: the layer has no down projection of its own and reads the cache rows of an earlier run entry (the run list's
 `cache_of`) as they are stored, with its own up projections, queries, window and sink.
@@ -45,7 +45,7 @@ DEFAULT_NAMES = {"sink": "sink", "q": "q_proj.weight", "q_down": "q_down.weight"
 @register(MIXERS, "latent_attention")
 class LatentAttention(Mixer):
     """params: hidden_size, num_heads, plain_dim, rot_dim, value_dim, kv_rank, q_rank (0: queries straight from the
-    input), gate (bool: sigmoid output gate), position (PartSpec of a rotary encoding over rot_dim), scale, eps,
+    input), gate (False, True: a sigmoid output gate per value, "head": one per head), position (PartSpec of a rotary encoding over rot_dim), scale, eps,
     window (None or int: the keys a query keeps in sight), sink (bool: a learned softmax sink per head), shared_kv (bool:
     no down projection, the cache rows of another run entry), names (local tensor names of q, q_down, q_norm, q_up,
     kv_down, kv_norm, k_up, v_up, gate, out, sink)."""
@@ -63,6 +63,7 @@ class LatentAttention(Mixer):
         self.kv_rank = int(spec["kv_rank"])
         self.q_rank = int(spec.get("q_rank") or 0)
         self.gate = bool(spec.get("gate", False))
+        self.gate_per = self.vdim if spec.get("gate") == "head" else 1      # neighbouring values that share a gate
         self.scale = float(spec["scale"])
         self.eps = float(spec["eps"])
         self.window = spec.get("window")
@@ -74,8 +75,8 @@ class LatentAttention(Mixer):
         if self.rot % 2 or getattr(self.position, "dim", self.rot) != self.rot:
             raise ValueError("the rotated part must be even and as wide as the position encoding turns")
         self.row = -(-(self.kv_rank + self.rot) // ROW_STEP) * ROW_STEP
-        if self.row > 256:
-            raise ValueError(f"kv_rank + rot_dim = {self.kv_rank + self.rot} is not supported: cache rows are at most 256 wide")
+        if self.row > kernels.ATTENTION_MAX_HEAD_DIM:
+            raise ValueError(f"kv_rank + rot_dim = {self.kv_rank + self.rot} is not supported: cache rows are at most {kernels.ATTENTION_MAX_HEAD_DIM} wide")
         self.head_w = self.plain + self.rot
 
     # ---------------------------------------------------------------- tensors
@@ -96,7 +97,7 @@ class LatentAttention(Mixer):
         else:
             needs[n["q"]] = TensorNeed((H * self.head_w, self.hidden))
         if self.gate:
-            needs[n["gate"]] = TensorNeed((H * self.vdim, self.hidden))
+            needs[n["gate"]] = TensorNeed((H * self.vdim // self.gate_per, self.hidden))
         return needs
 
     def load(self, tensors):
@@ -165,12 +166,12 @@ class LatentAttention(Mixer):
         mixed = paged_attention(ctx.plan_for(self), q_rows, cache.k, cache.k, cache, ctx, H, 1, self.scale, self.window, sink=self.sink)
         if few:      # W_vup_h (weighted sum of latents), gate and rounding in one row kernel
             values = kernels.latent_values(mixed, self.v_up, proj if self.gate else None, self.gate_col,
-                                           torch.empty((tokens, H * self.vdim), dtype=self.dtype, device=device))
+                                           torch.empty((tokens, H * self.vdim), dtype=self.dtype, device=device), per=self.gate_per)
             return linear_to_stream(values, self.o, h)
         values = torch.empty((tokens, H, self.vdim), dtype=torch.float32, device=device)
         kernels.gemm_heads(mixed, self.v_up, values, w_is_nk=True)             # W_vup_h (weighted sum of latents)
         values = values.view(tokens, H * self.vdim)
         if self.gate or self.dtype != torch.float32:
             values = kernels.latent_gate(values, proj if self.gate else None, self.gate_col,
-                                         torch.empty((tokens, H * self.vdim), dtype=self.dtype, device=device))
+                                         torch.empty((tokens, H * self.vdim), dtype=self.dtype, device=device), per=self.gate_per)
         return linear_to_stream(values, self.o, h)

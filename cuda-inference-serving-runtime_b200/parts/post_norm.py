@@ -1,4 +1,5 @@
-"""Sub-blocks with a norm before and after: x <- x + s * norm_out(sub_block(norm_in(x))), s one factor per channel.
+"""Sub-blocks with a norm after, and most with one before: x <- x + s * norm_out(sub_block(norm_in(x))), s one factor per
+channel; without a norm before, the sub-block reads the stream itself.
 
 The whole seam between two sub-blocks is one kernel (`kernels.post_norm`): a sub-block's output stays pending in the stream
 object, with its output norm, until the next sub-block (or the final norm) asks for its normed input; the kernel then norms the
@@ -59,20 +60,22 @@ class PostNormStream:
         return {"y": self.pending, "post_w": weight, "post_eps": eps, "post_kind": kind}
 
     def read(self, norm, dtype: torch.dtype, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """Bring everything pending into the stream and return its norm in `dtype`; `rows` picks tokens, and the stream is
-        then left as it is."""
+        """Bring everything pending into the stream and return its norm in `dtype` (norm None: the stream itself); `rows`
+        picks tokens, and the stream is then left as it is."""
         n = self.x.shape[0] if rows is None else rows.numel()
-        h = torch.empty((n, self.x.shape[1]), dtype=dtype, device=self.x.device)
+        as_it_is = norm is None and rows is None and dtype == self.x.dtype      # no copy: what reads it is done before the next write
+        h = None if as_it_is else torch.empty((n, self.x.shape[1]), dtype=dtype, device=self.x.device)
         changed = self.pending is not None or self.extra is not None or self.vector is not None
         x_out = None
         if rows is None and changed:
             x_out = torch.empty_like(self.x) if self.x is self.embedded else self.x
-        kernels.post_norm(self.x, **self._pending(), extra=self.extra, vector=self.vector, x_out=x_out, pre_w=float_weight(norm),
-                          pre_eps=norm.eps, pre_kind=norm.kind, h=h, rows=rows)
+        if x_out is not None or h is not None:
+            pre = {"pre_kind": "none"} if norm is None else {"pre_w": float_weight(norm), "pre_eps": norm.eps, "pre_kind": norm.kind}
+            kernels.post_norm(self.x, **self._pending(), extra=self.extra, vector=self.vector, x_out=x_out, **pre, h=h, rows=rows)
         if x_out is not None:
             self.x = x_out
             self.pending = self.pending_norm = self.extra = self.vector = None
-        return h
+        return self.x if as_it_is else h
 
     def finish(self, norm, dtype: torch.dtype, rows: torch.Tensor) -> torch.Tensor:
         """The model's last step: the normed stream at the wanted rows."""
@@ -87,14 +90,15 @@ class PostNormStream:
 
 @register(ARRANGEMENTS, "pre_post_norm_scaled")
 class PrePostNormBlock:
-    """x += s1 * norm1b(mixer(norm1(x))); x += s2 * norm2b(feed_forward(norm2(x))); the feed-forward half may be absent.  The
+    """x += s1 * norm1b(mixer(norm1(x))); x += s2 * norm2b(feed_forward(norm2(x))); the feed-forward half may be absent, and so
+    may the norms ahead (`mixer_norm`, `feed_forward_norm` None: the sub-block reads the stream itself).  The
     layer's `extras` give the output norms ("mixer_out_norm", "feed_forward_out_norm") and, where a layer has them, the
     scales ("mixer_scale", "feed_forward_scale": `ChannelScale`).  Norms name their kind (layer_norm, rms_norm)."""
 
     def __init__(self, spec: LayerSpec, dtype: torch.dtype):
         self.spec = spec
         self.dtype = dtype
-        norm = lambda part: build_part(NORMS, part, dtype, "norm")
+        norm = lambda part: None if part is None else build_part(NORMS, part, dtype, "norm")
         scale = lambda name: ChannelScale(spec.extras[name], dtype) if name in spec.extras else None
         self.mixer_norm, self.mixer_out_norm = norm(spec.mixer_norm), norm(spec.extras["mixer_out_norm"])
         self.mixer = build_part(MIXERS, spec.mixer, dtype, "mixer")

@@ -64,10 +64,14 @@ def scaled_frequencies(freq: torch.Tensor, theta: float, dim: int, scaling) -> t
     lo = max(floor(pair(fast)), 0) and hi = min(ceil(pair(slow)), dim - 1), pairs up to lo keep their frequency, pairs
     from hi on are slowed by `factor`, and those between are blended linearly:
     ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), f_i' = f_i / factor * ramp_i + f_i * (1 - ramp_i).
-    Both cos and sin are multiplied by 0.1 ln(factor) + 1."""
+    Both cos and sin are multiplied by 0.1 ln(factor) + 1.
+
+    kind "linear" (factor): every frequency is divided by `factor`."""
     import math
 
     kind = scaling.get("kind", "yarn")
+    if kind == "linear":
+        return freq / float(scaling["factor"]), 1.0
     if kind == "wavelength":
         return frequencies_by_wavelength(freq, scaling), 1.0
     if kind != "yarn":

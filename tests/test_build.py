@@ -11,7 +11,7 @@ def names(source):
 def test_the_include_closure_follows_every_kind_of_included_file():
     # a .cu file that includes another .cu file and a .h beside the .cuh headers
     assert names("attention_static_scratch.cu") == ["attention.cu", "attention_static_scratch.cu", "attention_static_scratch.h",
-                                                    "common.cuh"]
+                                                    "common.cuh", "softcap.cuh"]
     # headers included by headers
     assert {"tcgen05.cuh", "tma.cuh", "common.cuh"} <= set(names("gemm_tcgen05.cu"))
     assert names("elementwise.cu") == ["common.cuh", "elementwise.cu"]

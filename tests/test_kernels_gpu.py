@@ -455,7 +455,7 @@ def test_unsupported_head_size_is_refused_clearly():
     with pytest.raises(k.KernelError, match="multiples of 16"):
         k.attention_library(40, torch.float32)
     with pytest.raises(k.KernelError, match="multiples of 16"):
-        k.attention_library(272, torch.bfloat16)
+        k.attention_library(528, torch.bfloat16)
 
 
 @pytest.mark.parametrize("m", [1, 5, 8, 9, 16, 33, 64])
