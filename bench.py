@@ -27,12 +27,14 @@ every request holding about 4096 tokens of context while it decodes.  Prints ONE
 --workload mixed: the continuous-batching workload (by default the SmolLM2-1.7B sizes, 64 requests with prompts
 of 128 to 2048 tokens, 256 generated tokens each) through the scheduler with graphs on; prints total, prefill
 and decode tokens per second, launch counts, graph statistics and a roofline for the whole run.
---designs SIZES [--design zurolorn|ronolorn|gipozen|vilodra|kezunex]: Zurolorn (latent attention, routed experts), Ronolorn (windowed
+--designs SIZES [--design zurolorn|ronolorn|gipozen|vilodra|kezunex|tekezen]: Zurolorn (latent attention, routed experts), Ronolorn (windowed
 attention, gated delta rule, several residual streams), Gipozen (differential attention with convolved projections,
 depth-weighted average of the stream, PolyNorm and routed gated feed-forwards), Vilodra (lightning attention with a state
-per head, differential attention with rotary positions, windowed latent attention with sinks, gelu experts) or Kezunex
+per head, differential attention with rotary positions, windowed latent attention with sinks, gelu experts), Kezunex
 (softmax attention beside a state-space mixer, real-gated linear recurrence, matrix memory; the designs whose kernels are
-most like its own, Ronolorn and Vilodra, stand beside it too) beside the Llama shape of equal size at the named widths:
+most like its own, Ronolorn and Vilodra, stand beside it too) or Tekezen (windowed latent attention with a gate per head,
+windowed grouped attention with kept first tokens and bent scores, clamped gated feed-forwards, norms on outputs only, a
+table of token pairs; Vilodra and Gipozen beside it too) beside the Llama shape of equal size at the named widths:
 prompt and decode tokens per second of each, and per kind of kernel the device time and the distance from the roofline.
 --impl reference: the reference's own stock code on the same decode workload (see reference_arm).
 
@@ -539,13 +541,36 @@ def kezunex_pair(width: int, layers: int, heads: int, ff_active: int, experts: i
             "vilodra": others["vilodra"]}
 
 
+def tekezen_pair(width: int, layers: int, heads: int, ff_active: int, experts: int = 0, top: int = 0, vocab: int = 32000):
+    """A Tekezen shape and the Llama shape of equal size beside it: the same width, layers, vocabulary and query heads of 64.
+    Even layers have latent attention (rows of 96 + 32, values of 64, windows of 1024 keys) and a dense feed-forward, odd ones
+    grouped attention with a quarter as many key heads (windows of 1024 keys with 64 kept first ones, scores bent at 20,
+    shared values) and `top` of `experts` experts beside a shared one, together as wide as the dense feed-forward; 65,521 buckets of token
+    pairs; the table is the head.  Vilodra and Gipozen, the designs with the like kernels, of the same sizes beside them."""
+    experts, top = max(experts, 4), max(top, 1)
+    yarn = {"base": 10000.0, "dims": 32, "scaling": {"factor": 4.0, "original": 2048, "fast": 16.0, "slow": 2.0}}
+    lat = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 96, "rot": yarn, "scale": 96 ** -0.5, "mask": {"size": 1024}}
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 20.0, "v_mix": True,
+           "mask": {"size": 1024, "keep_first": 64}, "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0}}}
+    ff = ff_active // (top + 1) // 64 * 64
+    dense = {"kind": "dense", "ff": ff_active, "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": top}, "shared": {"ff": ff, "limit": 7.0}}
+    teke = {"architecture": "Tekezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "max_positions": 8192,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 40503, "mul_cur": 17}},
+            "layers": [{"type": "attention", "mixer": att, "mlp": moe} if i % 2 else {"type": "latent_attention", "mixer": lat, "mlp": dense}
+                       for i in range(layers)]}
+    others = vilodra_pair(width, layers, heads, ff_active, experts, top, vocab)
+    return {"tekezen": teke, "llama": others["llama"], "vilodra": others["vilodra"],
+            "gipozen": gipozen_pair(width, layers, heads, ff_active, experts, top, vocab)[0]}
+
+
 DESIGN_SIZES = {"1024": (1024, 8, 16, 2048, 16, 4), "2048": (2048, 8, 32, 4096, 32, 4), "4096": (4096, 4, 32, 8192, 64, 8)}
 KERNEL_KIND = {   # which kernels of the two designs are alike
     "gemm_tcgen05": "product, many tokens", "gemm_library": "product, many tokens", "gemm_tcgen05_swiglu": "feed-forward product, many tokens",
     "gemm_tcgen05_rope": "product, many tokens", "gemm_tcgen05_grouped": "feed-forward product, many tokens",
     "gemm_tcgen05_grouped_gated": "feed-forward product, many tokens", "skinny_gemm": "product, few tokens",
     "moe_rows": "feed-forward product, few tokens", "gemm_heads": "product per head", "attn_prefill_wide": "prompt attention", "attn_prefill": "prompt attention",
-    "attn_decode": "decode attention", "merge_out_proj": "product, few tokens", "add_rmsnorm": "norm", "embedding": "row kernels", "rope_store": "row kernels",
+    "attn_decode": "decode attention", "merge_out_proj": "product, few tokens", "add_rmsnorm": "norm", "embedding": "row kernels", "embedding_pairs": "row kernels", "rope_store": "row kernels",
     "latent_rows": "row kernels", "latent_query": "row kernels", "latent_gate": "row kernels", "latent_absorb": "product per head",
     "latent_values": "product per head", "moe_select": "row kernels", "moe_gather": "row kernels",
     "moe_combine": "row kernels", "moe_sort": "bookkeeping", "stream_add": "row kernels", "swiglu": "row kernels",
@@ -673,7 +698,7 @@ def generic_need(name: str, shape: tuple, cache_tokens: int, causal: int):
     if name == "add_rmsnorm":
         rows, hidden, added = shape
         return rows * hidden * (4 + (8 if added else 0) + 2), 0.0
-    if name in ("embedding", "stream_add"):
+    if name in ("embedding", "embedding_pairs", "stream_add"):
         return shape[0] * shape[1] * 8, 0.0
     if name in ("latent_rows", "latent_query", "rope_store"):
         return shape[0] * shape[1] * 6, 0.0
@@ -747,7 +772,7 @@ def design_comparison(args, hbm_gbs: float, burst_tflops: float, peak_source: st
 
     sizes = [s for s in args.designs.split(",") if s]
     batch, context, prompt = args.batch, min(args.context, 2048), PREFILL_TOKENS
-    pair = {"ronolorn": ronolorn_pair, "gipozen": gipozen_pair, "vilodra": vilodra_pair, "kezunex": kezunex_pair}.get(args.design, design_pair)
+    pair = {"ronolorn": ronolorn_pair, "gipozen": gipozen_pair, "vilodra": vilodra_pair, "kezunex": kezunex_pair, "tekezen": tekezen_pair}.get(args.design, design_pair)
     line = {"designs": f"{args.design} beside llama at equal size", "dtype": "bf16", "data": "synthetic token ids, seeded random weights",
             "batch": batch, "context": context, "prompt_tokens": prompt, "peaks": peak_source, "sizes": {}}
     sampler = ClockSampler().start()
@@ -1011,12 +1036,14 @@ def main() -> int:
     parser.add_argument("--designs", metavar="SIZES", default=None,
                         help="instead of the default workload: Zurolorn beside the Llama shape of equal size, prompt and decode, at "
                              "the named widths (comma-separated, from 1024, 2048, 4096)")
-    parser.add_argument("--design", choices=["zurolorn", "ronolorn", "gipozen", "vilodra", "kezunex"], default="zurolorn",
+    parser.add_argument("--design", choices=["zurolorn", "ronolorn", "gipozen", "vilodra", "kezunex", "tekezen"], default="zurolorn",
                         help="--designs: which design stands beside the Llama shape (ronolorn: windowed attention, gated delta rule, "
                              "four residual streams, dense feed-forward; gipozen: differential attention, depth-weighted average, "
                              "PolyNorm and routed gated feed-forwards; vilodra: lightning attention, differential attention with "
                              "rotary positions, windowed latent attention with sinks, dense gated and routed gelu feed-forwards; "
-                             "kezunex: softmax attention beside a state-space mixer, real-gated linear recurrence, matrix memory)")
+                             "kezunex: softmax attention beside a state-space mixer, real-gated linear recurrence, matrix memory; "
+                             "tekezen: windowed latent attention with a gate per head, windowed grouped attention with kept first "
+                             "tokens and bent scores, clamped gated feed-forwards)")
     args = parser.parse_args()
     if args.workload == "mixed" and "--preset" not in " ".join(sys.argv):
         args.preset = "smollm2-1.7b"

@@ -36,6 +36,27 @@ __device__ __forceinline__ float turned(const float* head, const float* w, float
     return v;
 }
 
+// Coordinates d .. d + 3 of a head whose weight is in the row already (times the common factor inv), pairs across the halves,
+// d, rot_half and the head's place in the row multiples of four: all four lie in the same half, and so do their partners.
+__device__ __forceinline__ float4 turned_four(const float* head, float inv, int d, int rot_half, const float* cs, const float* sn) {
+    const float4 x = *reinterpret_cast<const float4*>(head + d);
+    if (d >= 2 * rot_half) return make_float4(x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+    const bool first = d < rot_half;
+    const int f = first ? d : d - rot_half;
+    const float4 y = *reinterpret_cast<const float4*>(head + (first ? d + rot_half : f));
+    const float4 c = *reinterpret_cast<const float4*>(cs + f), s = *reinterpret_cast<const float4*>(sn + f);
+    const float sign = first ? -inv : inv;
+    return make_float4(x.x * inv * c.x + sign * y.x * s.x, x.y * inv * c.y + sign * y.y * s.y, x.z * inv * c.z + sign * y.z * s.z,
+                       x.w * inv * c.w + sign * y.w * s.w);
+}
+__device__ __forceinline__ void store_four(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* dst, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 raw;
+    raw.x = *reinterpret_cast<const uint32_t*>(&lo); raw.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = raw;
+}
+
 // Coordinates d and d + 1 (d even) of a head after norm and rotation.  Neighbouring pairs turn together, so one pair of
 // table entries serves both; the other pairing takes each coordinate's partner from across the head.
 __device__ __forceinline__ float2 turned_pair(const float* head, const float* w, float inv, int d, int width, int rot_half,
@@ -60,33 +81,70 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
                       const int* __restrict__ block_table, int table_width, int page_size, int hq, int hkv, int key_dim,
                       int value_dim, int D, int n_cols, int per_head, float temp_coef, double temp_every,
                       const float* __restrict__ v_other, int other_stride, float blend) {
-    extern __shared__ float row[];            // n_cols floats: the token's projection with its bias
-    __shared__ float scratch[32];
+    extern __shared__ __align__(16) float row[];            // n_cols floats: the token's projection with its bias
+    __shared__ float scratch[64];
     pdl_trigger();
     const int t = blockIdx.x;
     const int pos = positions[t];
     const int slot = req_slot[token_req[t]];
     pdl_wait();
     const float* src = proj + (size_t)t * row_stride;
-    for (int i = threadIdx.x; i < n_cols; i += blockDim.x) row[i] = src[i] + (bias ? bias[i] : 0.f);
-    if (v_other) {       // a thread blends the columns it has just brought in
-        const float* other = v_other + (size_t)t * other_stride;
-        const int v_end = v_col + hkv * value_dim;
-        for (int i = threadIdx.x; i < v_end; i += blockDim.x)
-            if (i >= v_col) row[i] = (1.f - blend) * row[i] + blend * other[i - v_col];
+    const int nq = hq * key_dim, nk = hkv * key_dim, k_end = k_col + nk;
+    const bool whole = !per_head && (q_norm || k_norm);
+    // the norms' weights join the row as it comes in, unless the values are the keys as projected
+    const bool weighted = whole && v_col >= 0;
+    // runs of four columns that lie in one projection (and one head) each
+    const bool wide = !((row_stride | k_col | k_end | n_cols | key_dim | value_dim) & 3) && v_col >= 0 && !(v_col & 3) && !bias && !per_head
+                      && !(reinterpret_cast<uintptr_t>(proj) & 15)
+                      && !((reinterpret_cast<uintptr_t>(q_norm) | reinterpret_cast<uintptr_t>(k_norm)) & 15);
+    const float* other = v_other ? v_other + (size_t)t * other_stride : nullptr;
+    float sq_q = 0.f, sq_k = 0.f;
+    if (wide) {
+        for (int i = threadIdx.x; i < n_cols / 4; i += blockDim.x) {
+            const int col = 4 * i;
+            float4 x = reinterpret_cast<const float4*>(src)[i];
+            const float sq = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+            const float* w = nullptr;
+            if (col < nq) { sq_q += sq; w = q_norm ? q_norm + col : nullptr; }
+            else if (col >= k_col && col < k_end) { sq_k += sq; w = k_norm ? k_norm + (col - k_col) : nullptr; }
+            if (w) {
+                const float4 f = *reinterpret_cast<const float4*>(w);
+                x.x *= f.x; x.y *= f.y; x.z *= f.z; x.w *= f.w;
+            } else if (other && col >= v_col) {
+                const float* o = other + (col - v_col);
+                x.x = (1.f - blend) * x.x + blend * o[0]; x.y = (1.f - blend) * x.y + blend * o[1];
+                x.z = (1.f - blend) * x.z + blend * o[2]; x.w = (1.f - blend) * x.w + blend * o[3];
+            }
+            reinterpret_cast<float4*>(row)[i] = x;
+        }
+    } else {
+        for (int i = threadIdx.x; i < n_cols; i += blockDim.x) {
+            float x = src[i] + (bias ? bias[i] : 0.f);
+            if (i < nq) {
+                sq_q += x * x;
+                if (weighted && q_norm) x *= q_norm[i];
+            } else if (i >= k_col && i < k_end) {
+                sq_k += x * x;
+                if (weighted && k_norm) x *= k_norm[i - k_col];
+            } else if (other && i >= v_col) {
+                x = (1.f - blend) * x + blend * other[i - v_col];
+            }
+            row[i] = x;
+        }
     }
-    __syncthreads();
-    const int nq = hq * key_dim, nk = hkv * key_dim;
     float inv_q = 1.f, inv_k = 1.f;
-    if (q_norm && !per_head) {
-        float sq = 0.f;
-        for (int i = threadIdx.x; i < nq; i += blockDim.x) sq += row[i] * row[i];
-        inv_q = 1.f / sqrtf(block_sum(sq, scratch) / (float)nq + eps);
-    }
-    if (k_norm && !per_head) {
-        float sq = 0.f;
-        for (int i = threadIdx.x; i < nk; i += blockDim.x) sq += row[k_col + i] * row[k_col + i];
-        inv_k = 1.f / sqrtf(block_sum(sq, scratch) / (float)nk + eps);
+    if (whole) {       // both sums in one pass over the block, in the fixed order of block_sum
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = (blockDim.x + 31) >> 5;
+        sq_q = warp_sum(sq_q);
+        sq_k = warp_sum(sq_k);
+        if (lane == 0) { scratch[warp] = sq_q; scratch[32 + warp] = sq_k; }
+        __syncthreads();
+        sq_q = warp_sum(lane < n_warps ? scratch[lane] : 0.f);
+        sq_k = warp_sum(lane < n_warps ? scratch[32 + lane] : 0.f);
+        if (q_norm) inv_q = 1.f / sqrtf(sq_q / (float)nq + eps);
+        if (k_norm) inv_k = 1.f / sqrtf(sq_k / (float)nk + eps);
+    } else {
+        __syncthreads();
     }
     const float* cs = cos_t ? cos_t + (size_t)t * rot_half : nullptr;
     const float* sn = sin_t ? sin_t + (size_t)t * rot_half : nullptr;
@@ -98,9 +156,28 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
         return 1.f / sqrtf(warp_sum(sq) / (float)key_dim + eps);
     };
     const float temp = temp_coef != 0.f ? 1.f + temp_coef * logf((float)(floor((double)(pos + 1) / temp_every) + 1.0)) : 1.f;
+    if (wide && !interleaved && !(rot_half & 3) && !((reinterpret_cast<uintptr_t>(cos_t) | reinterpret_cast<uintptr_t>(sin_t)) & 15)) {
+        // four coordinates per thread, the heads of queries, keys and values one after the other
+        const int per = D >> 2;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int i = threadIdx.x; i < hq * per; i += blockDim.x) {
+            const int h = i / per, d = 4 * (i - h * per);
+            store_four(q_out + (size_t)t * hq * D + 4 * i, d < key_dim ? turned_four(row + h * key_dim, temp * inv_q, d, rot_half, cs, sn) : zero);
+        }
+        if (!k_cache) return;
+        const int page = block_table[(size_t)slot * table_width + pos / page_size];
+        if (page < 0) return;                 // the host reserves a page before every write; never follow a missing entry
+        for (int i = threadIdx.x; i < hkv * per; i += blockDim.x) {
+            const int g = i / per, d = 4 * (i - g * per);
+            const size_t dst = (((size_t)page * hkv + g) * page_size + pos % page_size) * D + d;
+            store_four(k_cache + dst, d < key_dim ? turned_four(row + k_col + g * key_dim, inv_k, d, rot_half, cs, sn) : zero);
+            store_four(v_cache + dst, d < value_dim ? *reinterpret_cast<const float4*>(row + v_col + g * value_dim + d) : zero);
+        }
+        return;
+    }
     for (int h = warp; h < hq; h += n_warps) {
         const float inv = temp * (q_norm && per_head ? head_inv(row + h * key_dim) : inv_q);
-        const float* w = q_norm ? q_norm + (per_head ? 0 : h * key_dim) : nullptr;
+        const float* w = q_norm && !weighted ? q_norm + (per_head ? 0 : h * key_dim) : nullptr;
         for (int d = 2 * lane; d < D; d += 64)
             store_pair(q_out + ((size_t)t * hq + h) * D + d, turned_pair(row + h * key_dim, w, inv, d, key_dim, rot_half, interleaved, cs, sn));
     }
@@ -110,7 +187,7 @@ attention_rows_kernel(const float* __restrict__ proj, int row_stride, int k_col,
     const int off = pos % page_size;
     for (int g = warp; g < hkv; g += n_warps) {
         const float inv = k_norm && per_head ? head_inv(row + k_col + g * key_dim) : inv_k;
-        const float* w = k_norm ? k_norm + (per_head ? 0 : g * key_dim) : nullptr;
+        const float* w = k_norm && !weighted ? k_norm + (per_head ? 0 : g * key_dim) : nullptr;
         for (int d = 2 * lane; d < D; d += 64) {
             const float* vs = v_col >= 0 ? row + v_col + g * value_dim : row + k_col + g * key_dim;
             const size_t dst = (((size_t)page * hkv + g) * page_size + off) * D + d;

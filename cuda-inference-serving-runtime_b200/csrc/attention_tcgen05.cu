@@ -252,7 +252,10 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const uint32_t tmem_own = tmem_o + lane_base + (uint32_t)(group * D);     // this thread's row of its group's accumulator
         const float scale2 = SOFTCAP ? 1.f : scale * LOG2E;        // bent scores come in base-2 units
         auto softmax_sync = [&]() { asm volatile("bar.sync 1, %0;" ::"n"(SOFTMAX_THREADS) : "memory"); };
-        float m_used = -INFINITY, l = 0.f;
+        // bent scores lie in (-cap, cap): where 2^(cap log2 e) is far from a float's range they need no running max, and
+        // every exponential is taken against 0
+        const bool bounded = SOFTCAP && softcap * LOG2E <= 60.f;
+        float m_used = bounded ? 0.f : -INFINITY, l = 0.f;
         bool ok = true;
         uint32_t raw[HALF];
         auto step = [&](int j) {
@@ -271,7 +274,14 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (SOFTCAP) {
                     const Bend bend(scale, softcap);
 #pragma unroll
-                    for (int c = 0; c < HALF; ++c) raw[c] = __float_as_uint(bend(__uint_as_float(raw[c])));
+                    for (int c = 0; c < HALF; c += 4) {
+                        float x[4];
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) x[e] = __uint_as_float(raw[c + e]);
+                        bend.four(x[0], x[1], x[2], x[3]);
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) raw[c + e] = __float_as_uint(x[e]);
+                    }
                 }
                 if (edge) {
 #pragma unroll
@@ -313,7 +323,7 @@ attn_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const float m_tile = mx * scale2;                     // the scale is positive: the max of the raw scores, scaled
             // the max in use moves only when it lags by more than RESCALE_STEP; the first finite max is taken as it is
             float alpha = 1.f;
-            const bool moved = m_tile > m_used + RESCALE_STEP || (m_used == -INFINITY && m_tile > -INFINITY);
+            const bool moved = bounded ? false : m_tile > m_used + RESCALE_STEP || (m_used == -INFINITY && m_tile > -INFINITY);
             if (moved) {
                 alpha = m_used == -INFINITY ? 0.f : fast_exp2(m_used - m_tile);
                 m_used = m_tile;

@@ -40,6 +40,13 @@ CISR_EXPORT int cisr_embedding(const void* table, int table_dtype, const int* id
     return launch_kernel(embedding_kernel<float>, dim3(tokens), dim3(128), 0, s, g_pdl, (const float*)table, ids, out, hidden, vocab, scale);
 }
 
+__device__ __forceinline__ float4 load_four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load_four(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
 // The same with a second table, looked up by a hash of the token and the one before it in its sequence:
 //   out[t] = table[id] * scale + pairs[(before * mul_prev + id * mul_cur) mod buckets],
 // or, for a sequence's first token, the row behind the buckets.  The token before comes from the step itself, or, for
@@ -77,6 +84,13 @@ __global__ void embedding_pairs_kernel(const TT* __restrict__ table, const TT* _
     const TT* src = table + (size_t)id * hidden;
     const TT* add = pairs + (size_t)bucket * hidden;
     float* dst = out + (size_t)t * hidden;
+    if (!(hidden & 3) && !((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(pairs) | reinterpret_cast<uintptr_t>(out)) & 15)) {
+        for (int d = 4 * threadIdx.x; d < hidden; d += 4 * blockDim.x) {
+            const float4 a = load_four(src + d), b = load_four(add + d);
+            *reinterpret_cast<float4*>(dst + d) = make_float4(a.x * scale + b.x, a.y * scale + b.y, a.z * scale + b.z, a.w * scale + b.w);
+        }
+        return;
+    }
     for (int d = threadIdx.x; d < hidden; d += blockDim.x) dst[d] = to_float(src[d]) * scale + to_float(add[d]);
 }
 
@@ -87,7 +101,7 @@ CISR_EXPORT int cisr_embedding_pairs(const void* table, const void* pairs, int t
     if (tokens <= 0) return 0;
     if (buckets <= 0 || mul_prev < 0 || mul_prev >= buckets || mul_cur < 0 || mul_cur >= buckets) return -2;
     cudaStream_t s = (cudaStream_t)stream;
-    const dim3 block(hidden >= 2048 ? 512 : 128);
+    const dim3 block(hidden >= 2048 ? 256 : 128);
     if (table_dtype == CISR_BF16)
         return launch_kernel(embedding_pairs_kernel<__nv_bfloat16>, dim3(tokens), block, 0, s, g_pdl, (const __nv_bfloat16*)table,
                              (const __nv_bfloat16*)pairs, ids, positions, token_req, req_slot, q_start, q_len, last, out, hidden, vocab, scale,

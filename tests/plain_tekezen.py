@@ -91,11 +91,9 @@ def turn_halves(x: torch.Tensor, freq: torch.Tensor, magnitude: float = 1.0) -> 
 # ------------------------------------------------------------------ softmax over the keys in sight
 def in_sight(T: int, window=None, keep_first: int = 0) -> torch.Tensor:
     """see[i, j]: j is not behind i, and is one of the last `window` keys or one of the sequence's first `keep_first`."""
-    see = torch.zeros(T, T, dtype=torch.bool)
-    for i in range(T):
-        for j in range(i + 1):
-            see[i, j] = window is None or i - j < window or j < keep_first
-    return see
+    i, j = torch.arange(T)[:, None], torch.arange(T)[None, :]
+    see = j <= i
+    return see if window is None else see & ((i - j < window) | (j < keep_first))
 
 
 def softmax_rows(scores: torch.Tensor, see: torch.Tensor) -> torch.Tensor:

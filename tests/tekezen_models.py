@@ -135,11 +135,14 @@ def tensor_shapes(cfg: dict) -> dict:
     return shapes
 
 
-def make_weights(cfg: dict, seed: int, gain: float = 1.0) -> dict:
+def make_weights(cfg: dict, seed: int, gain: float = 1.0, calm: bool = False) -> dict:
     """Seeded weights, every value representable in bfloat16 (so a bfloat16 engine and a float oracle start alike).
     `gain` scales the queries (of the grouped attention through the weight of their norm): a larger one makes the softmax
     peaked.  Norm weights, gates, routers and feed-forwards are spread widely, so that leaving one out, or a limit, or using
-    an offset without its one, moves the logits."""
+    an offset without its one, moves the logits.  `calm`: flatter softmaxes, gates and routers, for bfloat16 runs of whole
+    models: among hundreds of positions some have a sub-block whose output nearly cancels, and its norm magnifies the one
+    rounding of what the sub-block read (the plain implementation, given rounded inputs, strays as far there)."""
+    gain, spread = (0.5 * gain, 1.0 / 3.0) if calm else (gain, 1.0)
     rng = np.random.default_rng(seed)
     out = {}
     latent_layers = {f"l{i}." for i, spec in enumerate(cfg["layers"]) if spec["type"] == "latent_attention"}
@@ -152,15 +155,17 @@ def make_weights(cfg: dict, seed: int, gain: float = 1.0) -> dict:
         elif leaf == "vmix":
             value = 0.25 + 0.4 * rng.random()
         elif leaf == "router":
-            value = 1.5 / np.sqrt(shape[1]) * rng.standard_normal(shape)
+            value = 1.5 * spread / np.sqrt(shape[1]) * rng.standard_normal(shape)
         elif name == "embed":
             value = rng.standard_normal(shape)
         elif name == "bigram":
             value = 0.8 * rng.standard_normal(shape)
         elif ".mix." in name and leaf == "q" and name[:name.index("mix.")] in latent_layers:
             value = gain / np.sqrt(shape[1]) * rng.standard_normal(shape)
-        elif leaf in ("g", "gate", "up"):
-            value = 1.5 * rng.standard_normal(shape) / np.sqrt(shape[-1])
+        elif leaf == "g":
+            value = 1.5 * spread * rng.standard_normal(shape) / np.sqrt(shape[-1])
+        elif leaf in ("gate", "up"):
+            value = (1.0 if calm else 1.5) * rng.standard_normal(shape) / np.sqrt(shape[-1])
         else:
             value = rng.standard_normal(shape) / np.sqrt(shape[-1])
         out[name] = torch.tensor(np.asarray(value), dtype=torch.float32).to(torch.bfloat16).to(torch.float64)
