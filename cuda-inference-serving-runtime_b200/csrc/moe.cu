@@ -134,23 +134,29 @@ moe_select_kernel(const float* __restrict__ logits, int tokens, int n_experts, i
             __syncwarp();
         }
     }
-    float chosen_sum = 0.f;                                          // lane 0's: the chosen scores, added best first
+    // Every lane follows the choice; lane k (mod 32) holds the k-th chosen score until the sum is known.
+    float chosen_sum = 0.f, mine = 0.f;                              // the sum is taken best first
+    float* w_out = weight + (size_t)t * top;
     for (int k = 0; k < top; ++k) {
         float v;
         int best = warp_best(rank, open_, n_experts, v);
         __syncwarp();
-        if (lane == 0) {
-            if (best == 0x7fffffff) best = 0;                        // fewer open experts than `top`: the host refuses such a configuration
-            else open_[best] = 0;
+        if (best == 0x7fffffff) best = 0;                            // fewer open experts than `top`: the host refuses such a configuration
+        const float s = score[best];
+        chosen_sum += s;
+        if (lane == (k & 31)) {
+            mine = s;
+            open_[best] = 0;
             chosen[(size_t)t * top + k] = best;
-            chosen_sum += score[best];
-            weight[(size_t)t * top + k] = renormalize ? score[best] : score[best] * route_scale;
+            if (top > 32) w_out[k] = renormalize ? s : s * route_scale;
         }
         __syncwarp();
     }
-    if (renormalize && lane == 0) {
-        const float den = chosen_sum + 1e-20f;
-        for (int k = 0; k < top; ++k) weight[(size_t)t * top + k] = weight[(size_t)t * top + k] / den * route_scale;
+    const float den = chosen_sum + 1e-20f;
+    if (top <= 32) {
+        if (lane < top) w_out[lane] = renormalize ? mine / den * route_scale : mine * route_scale;
+    } else if (renormalize) {
+        for (int k = lane; k < top; k += 32) w_out[k] = w_out[k] / den * route_scale;       // a lane's own writes
     }
 }
 
